@@ -65,6 +65,7 @@ def _register_builtin() -> None:
     from .bunudra import BunudraConfig
     from .dubazen import DubazenConfig
     from .ditilix import DitilixConfig
+    from .futepel import FutepelConfig
     from .lanilix import LanilixConfig
     from .qwen3 import Qwen3Config
     register_architecture(Qwen3Config.architecture, Qwen3Config, _decoder_model)
@@ -72,6 +73,7 @@ def _register_builtin() -> None:
     register_architecture(BunudraConfig.architecture, BunudraConfig, _decoder_model)
     register_architecture(DitilixConfig.architecture, DitilixConfig, _decoder_model)
     register_architecture(DubazenConfig.architecture, DubazenConfig, _decoder_model)
+    register_architecture(FutepelConfig.architecture, FutepelConfig, _decoder_model)
 
 
 _register_builtin()

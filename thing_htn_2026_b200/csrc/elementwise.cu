@@ -112,6 +112,134 @@ THN_API int thn_gather_rows_scaled(float* out, const void* table, const int* ind
     return thn_launch_status("gather_rows_scaled");
 }
 
+// out[m] = table[token] * scale + pairs[row of (token before, token)] + positions[pos]: the start of a
+// float32 residual stream.  The pair's row is (before * mul_before + token * mul_token) mod buckets; a
+// sequence's first token takes row `buckets`, the table's last.  The token before the first row that a
+// sequence brings is what its last step left in `previous`; the block of that row leaves the step's last
+// token there, after it has read (no other block touches the slot).  pairs and positions may be null.
+template <typename T>
+__global__ void embed_rows_kernel(float* __restrict__ out, const T* __restrict__ table, const int* __restrict__ tokens, int width,
+                                  int n_table_rows, float scale, const T* __restrict__ pairs, int buckets, long long mul_before,
+                                  long long mul_token, int* __restrict__ previous, const T* __restrict__ positions,
+                                  int n_positions, const int* __restrict__ row_slot, const int* __restrict__ row_pos,
+                                  const int* __restrict__ cu_seqlens, const int* __restrict__ seq_lens, int n_seqs,
+                                  int* __restrict__ err) {
+    pdl_launch_dependents();
+    pdl_wait();
+    __shared__ int pair_row;
+    const int m = blockIdx.x;
+    const int slot = row_slot[m];
+    int pos = row_pos[m], token = tokens[m];
+    if (token < 0 || token >= n_table_rows) {
+        if (threadIdx.x == 0 && err) atomicOr(err, THN_ERR_TOKEN_RANGE);
+        token = 0;
+    }
+    if (positions != nullptr && pos >= n_positions) {
+        if (threadIdx.x == 0 && err) atomicOr(err, THN_ERR_POSITION_RANGE);
+        pos = n_positions - 1;
+    }
+    if (pairs != nullptr && threadIdx.x == 0) {
+        const bool first = row_pos[m] == seq_lens[slot];
+        const int before = first ? previous[slot] : tokens[m - 1];
+        int row = buckets;
+        if (row_pos[m] > 0) {
+            const long long mixed = (long long)before * mul_before + (long long)token * mul_token;
+            row = (int)(((mixed % buckets) + buckets) % buckets);
+        }
+        pair_row = row;
+        if (first) {
+            int lo = 0, hi = n_seqs - 1;              // the sequence of row m: the last one that starts at or before it
+            while (lo < hi) {
+                const int mid = (lo + hi + 1) >> 1;
+                if (cu_seqlens[mid] <= m) lo = mid; else hi = mid - 1;
+            }
+            previous[slot] = tokens[cu_seqlens[lo + 1] - 1];
+        }
+    }
+    __syncthreads();
+    const T* src = table + (size_t)token * width;
+    const T* pair = pairs != nullptr ? pairs + (size_t)pair_row * width : nullptr;
+    const T* place = positions != nullptr ? positions + (size_t)pos * width : nullptr;
+    float* dst = out + (size_t)m * width;
+    for (int i = threadIdx.x; i < width; i += blockDim.x) {
+        float v = to_f32<T>(src[i]) * scale;
+        if (pair != nullptr) v += to_f32<T>(pair[i]);
+        if (place != nullptr) v += to_f32<T>(place[i]);
+        dst[i] = v;
+    }
+}
+
+// table [n_table_rows, width], pairs [buckets + 1, width] and positions [n_positions, width] of the
+// activation type; previous int32 [slots], read and updated; seq_lens: the tokens each slot held before
+// the step; the rows of sequence i are [cu_seqlens[i], cu_seqlens[i + 1]).
+THN_API int thn_embed_rows(float* out, const void* table, const int* tokens, int n_rows, int width, int n_table_rows, float scale,
+                           const void* pairs, int buckets, long long mul_before, long long mul_token, int* previous,
+                           const void* positions, int n_positions, const int* row_slot, const int* row_pos,
+                           const int* cu_seqlens, const int* seq_lens, int n_seqs, int dtype, int* err, cudaStream_t stream) {
+    THN_CHECK_ARG(n_rows >= 0 && width > 0 && n_table_rows > 0 && n_seqs >= 0, "embed_rows: bad sizes rows=%d width=%d table=%d",
+                  n_rows, width, n_table_rows);
+    THN_CHECK_ARG(pairs == nullptr || (buckets > 0 && previous != nullptr), "embed_rows: pairs need buckets and the tokens before");
+    THN_CHECK_ARG(positions == nullptr || n_positions > 0, "embed_rows: an empty table of positions");
+    if (n_rows == 0) return THN_OK;
+    if (dtype == THN_F32)
+        thn_launch(embed_rows_kernel<float>, n_rows, 256, 0, stream, out, (const float*)table, tokens, width, n_table_rows, scale,
+                   (const float*)pairs, buckets, mul_before, mul_token, previous, (const float*)positions, n_positions, row_slot,
+                   row_pos, cu_seqlens, seq_lens, n_seqs, err);
+    else if (dtype == THN_BF16)
+        thn_launch(embed_rows_kernel<__nv_bfloat16>, n_rows, 256, 0, stream, out, (const __nv_bfloat16*)table, tokens, width,
+                   n_table_rows, scale, (const __nv_bfloat16*)pairs, buckets, mul_before, mul_token, previous,
+                   (const __nv_bfloat16*)positions, n_positions, row_slot, row_pos, cu_seqlens, seq_lens, n_seqs, err);
+    else
+        THN_CHECK_ARG(false, "embed_rows: unknown dtype %d", dtype);
+    return thn_launch_status("embed_rows");
+}
+
+// out = max(z, 0)^2, entry by entry.
+template <typename T>
+__global__ void squared_relu_kernel(T* __restrict__ out, const T* __restrict__ z, long long n) {
+    pdl_launch_dependents();
+    pdl_wait();
+    const long long e = (long long)blockIdx.x * blockDim.x + threadIdx.x;
+    if (e >= n) return;
+    const float v = fmaxf(to_f32<T>(z[e]), 0.f);
+    out[e] = from_f32<T>(v * v);
+}
+
+// The same, eight bfloat16 entries per thread.
+__global__ void squared_relu_bf16_vec_kernel(__nv_bfloat16* __restrict__ out, const __nv_bfloat16* __restrict__ z, long long vecs) {
+    pdl_launch_dependents();
+    pdl_wait();
+    const long long e = (long long)blockIdx.x * blockDim.x + threadIdx.x;
+    if (e >= vecs) return;
+    const uint4 raw = reinterpret_cast<const uint4*>(z)[e];
+    const __nv_bfloat162* in = reinterpret_cast<const __nv_bfloat162*>(&raw);
+    uint4 packed;
+    __nv_bfloat162* o2 = reinterpret_cast<__nv_bfloat162*>(&packed);
+#pragma unroll
+    for (int j = 0; j < 4; ++j) {
+        const float2 v = __bfloat1622float2(in[j]);
+        const float a = fmaxf(v.x, 0.f), b = fmaxf(v.y, 0.f);
+        o2[j] = __floats2bfloat162_rn(a * a, b * b);
+    }
+    reinterpret_cast<uint4*>(out)[e] = packed;
+}
+
+THN_API int thn_squared_relu(void* out, const void* z, long long n, int dtype, cudaStream_t stream) {
+    THN_CHECK_ARG(n >= 0, "squared_relu: bad size");
+    if (n == 0) return THN_OK;
+    const unsigned blocks = (unsigned)((n + 255) / 256);
+    if (dtype == THN_BF16 && n % 8 == 0 && (((uintptr_t)out | (uintptr_t)z) & 15) == 0)
+        thn_launch(squared_relu_bf16_vec_kernel, (unsigned)((n / 8 + 255) / 256), 256, 0, stream, (__nv_bfloat16*)out,
+                   (const __nv_bfloat16*)z, n / 8);
+    else if (dtype == THN_F32)
+        thn_launch(squared_relu_kernel<float>, blocks, 256, 0, stream, (float*)out, (const float*)z, n);
+    else if (dtype == THN_BF16)
+        thn_launch(squared_relu_kernel<__nv_bfloat16>, blocks, 256, 0, stream, (__nv_bfloat16*)out, (const __nv_bfloat16*)z, n);
+    else
+        THN_CHECK_ARG(false, "squared_relu: unknown dtype %d", dtype);
+    return thn_launch_status("squared_relu");
+}
+
 // x[i] *= scale in place, float32: a constant factor on logits.
 __global__ void scale_f32_kernel(float* __restrict__ x, long long n, float scale) {
     pdl_launch_dependents();
@@ -128,17 +256,18 @@ THN_API int thn_scale_f32(float* x, long long n, float scale, cudaStream_t strea
     return thn_launch_status("scale_f32");
 }
 
-// out[m, i] = a[m, i] * logistic(g[m, i]): an output gate on a mixer's concatenated heads.  The
-// gate's rows are g_stride elements apart (it may be a slice of a wider projected row).
+// out[m, i] = a[m, i] * logistic(g[m, i / per]): an output gate on a mixer's concatenated heads, one
+// number per entry (per 1) or one for `per` neighbours (a gate per head).  The gate's rows are g_stride
+// elements apart (it may be a slice of a wider projected row).
 template <typename T>
 __global__ void logistic_gate_kernel(T* __restrict__ out, const T* __restrict__ a, const T* __restrict__ g,
-                                     long long g_stride, long long n, int width) {
+                                     long long g_stride, long long n, int width, int per) {
     pdl_launch_dependents();
     pdl_wait();
     const long long e = (long long)blockIdx.x * blockDim.x + threadIdx.x;
     if (e >= n) return;
     const long long m = e / width;
-    const float z = to_f32<T>(g[m * g_stride + (e - m * width)]);
+    const float z = to_f32<T>(g[m * g_stride + (e - m * width) / per]);
     out[e] = from_f32<T>(to_f32<T>(a[e]) / (1.0f + expf(-z)));
 }
 
@@ -164,12 +293,38 @@ __global__ void logistic_gate_bf16_vec_kernel(__nv_bfloat16* __restrict__ out, c
     *reinterpret_cast<uint4*>(out + row * width + c) = make_uint4(res[0], res[1], res[2], res[3]);
 }
 
-THN_API int thn_logistic_gate(void* out, const void* a, const void* g, long long g_stride, int n_rows, int width,
+// One gate for `per` neighbours, a multiple of eight of them.
+__global__ void logistic_head_gate_bf16_vec_kernel(__nv_bfloat16* __restrict__ out, const __nv_bfloat16* __restrict__ a,
+                                                   const __nv_bfloat16* __restrict__ g, long long g_stride, int width, int per) {
+    pdl_launch_dependents();
+    pdl_wait();
+    const int c = (blockIdx.x * blockDim.x + threadIdx.x) * 8;
+    if (c >= width) return;
+    const long long row = blockIdx.y;
+    const uint4 ra = *reinterpret_cast<const uint4*>(a + row * width + c);
+    const float d = 1.0f + expf(-__bfloat162float(g[row * g_stride + c / per]));
+    const __nv_bfloat162* in = reinterpret_cast<const __nv_bfloat162*>(&ra);
+    uint4 packed;
+    __nv_bfloat162* o2 = reinterpret_cast<__nv_bfloat162*>(&packed);
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+        const float2 x = __bfloat1622float2(in[i]);
+        o2[i] = __floats2bfloat162_rn(x.x / d, x.y / d);
+    }
+    *reinterpret_cast<uint4*>(out + row * width + c) = packed;
+}
+
+THN_API int thn_logistic_gate(void* out, const void* a, const void* g, long long g_stride, int n_rows, int width, int per,
                               int dtype, cudaStream_t stream) {
-    THN_CHECK_ARG(n_rows >= 0 && width > 0 && g_stride >= width, "logistic_gate: bad sizes");
+    THN_CHECK_ARG(n_rows >= 0 && width > 0 && per > 0 && width % per == 0 && g_stride >= width / per, "logistic_gate: bad sizes");
     const long long n = (long long)n_rows * width;
     if (n == 0) return THN_OK;
-    if (dtype == THN_BF16 && width % 8 == 0 && g_stride % 8 == 0 && n_rows <= 65535 &&
+    if (dtype == THN_BF16 && per % 8 == 0 && n_rows <= 65535 && ((((uintptr_t)out) | ((uintptr_t)a)) & 15) == 0) {
+        thn_launch(logistic_head_gate_bf16_vec_kernel, dim3((width / 8 + 127) / 128, n_rows), 128, 0, stream, (__nv_bfloat16*)out,
+                   (const __nv_bfloat16*)a, (const __nv_bfloat16*)g, g_stride, width, per);
+        return thn_launch_status("logistic_gate");
+    }
+    if (dtype == THN_BF16 && per == 1 && width % 8 == 0 && g_stride % 8 == 0 && n_rows <= 65535 &&
         ((((uintptr_t)out) | ((uintptr_t)a) | ((uintptr_t)g)) & 15) == 0) {
         thn_launch(logistic_gate_bf16_vec_kernel, dim3((width / 8 + 127) / 128, n_rows), 128, 0, stream, (__nv_bfloat16*)out,
                    (const __nv_bfloat16*)a, (const __nv_bfloat16*)g, g_stride, width);
@@ -178,10 +333,10 @@ THN_API int thn_logistic_gate(void* out, const void* a, const void* g, long long
     const unsigned blocks = (unsigned)((n + 255) / 256);
     if (dtype == THN_F32)
         thn_launch(logistic_gate_kernel<float>, blocks, 256, 0, stream, (float*)out, (const float*)a, (const float*)g,
-                   g_stride, n, width);
+                   g_stride, n, width, per);
     else if (dtype == THN_BF16)
         thn_launch(logistic_gate_kernel<__nv_bfloat16>, blocks, 256, 0, stream, (__nv_bfloat16*)out, (const __nv_bfloat16*)a,
-                   (const __nv_bfloat16*)g, g_stride, n, width);
+                   (const __nv_bfloat16*)g, g_stride, n, width, per);
     else
         THN_CHECK_ARG(false, "logistic_gate: unknown dtype %d", dtype);
     return thn_launch_status("logistic_gate");

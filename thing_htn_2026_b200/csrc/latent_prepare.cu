@@ -11,8 +11,8 @@
 //                    part] and the value, written to the paged cache (keys of plain + rot
 //                    entries, values of a size of their own).
 //
-// The rotation pairs entry 2i with entry 2i + 1 of the rotated part: (a, b) with angle t becomes
-// (a cos t - b sin t, b cos t + a sin t); cos and sin come from tables [positions, rot / 2]
+// The rotation pairs entry 2i with entry 2i + 1 of the rotated part (interleaved) or entry i with
+// entry i + rot / 2 (half): (a, b) with angle t becomes (a cos t - b sin t, b cos t + a sin t); cos and sin come from tables [positions, rot / 2]
 // (which may carry a common magnitude).  float32 between the load and the one rounding at the
 // store; what is only copied is copied as it is.  One block per row.
 #include "common.cuh"
@@ -42,7 +42,7 @@ __global__ void __launch_bounds__(256) latent_assemble_kernel(
     T* __restrict__ q_out, const T* __restrict__ q_src, long long q_stride, const T* __restrict__ shared_src,
     long long shared_stride, const T* __restrict__ up, const float* __restrict__ cos_tab,
     const float* __restrict__ sin_tab, int table_len, const int* __restrict__ row_slot, const int* __restrict__ row_pos,
-    PagedKV kv, int n_heads, int plain, int rot, int value_src, int* __restrict__ err) {
+    PagedKV kv, int n_heads, int plain, int rot, int interleaved, int value_src, int* __restrict__ err) {
     pdl_launch_dependents();
     pdl_wait();
     const int m = blockIdx.x;
@@ -61,6 +61,8 @@ __global__ void __launch_bounds__(256) latent_assemble_kernel(
     const T* k_shared = shared_src + (size_t)m * shared_stride;
     const T* up_row = up + (size_t)m * n_heads * (plain + value_src);
     T* cache = (T*)kv.base;
+    // pair i of a rotated part: its first entry, and how far behind it the second one lies
+    const int first = interleaved ? 2 : 1, apart = interleaved ? 1 : half;
 
     // queries: the plain part as it is, the rest rotated
     for (int e = threadIdx.x; e < n_heads * plain; e += blockDim.x) {
@@ -69,11 +71,12 @@ __global__ void __launch_bounds__(256) latent_assemble_kernel(
     }
     for (int e = threadIdx.x; e < n_heads * half; e += blockDim.x) {
         const int h = e / half, i = e - h * half;
-        const float a = to_f32<T>(q_row[h * D + plain + 2 * i]), b = to_f32<T>(q_row[h * D + plain + 2 * i + 1]);
+        const T* src = q_row + h * D + plain + first * i;
+        const float a = to_f32<T>(src[0]), b = to_f32<T>(src[apart]);
         const float c = c_row[i], s = s_row[i];
-        T* dst = q_out + ((size_t)m * n_heads + h) * D + plain + 2 * i;
+        T* dst = q_out + ((size_t)m * n_heads + h) * D + plain + first * i;
         dst[0] = from_f32<T>(a * c - b * s);
-        dst[1] = from_f32<T>(b * c + a * s);
+        dst[apart] = from_f32<T>(b * c + a * s);
     }
     if (page < 0) return;
     // keys: every head's plain part from the up-projection, then the shared part, rotated
@@ -83,11 +86,11 @@ __global__ void __launch_bounds__(256) latent_assemble_kernel(
     }
     for (int e = threadIdx.x; e < n_heads * half; e += blockDim.x) {
         const int h = e / half, i = e - h * half;
-        const float a = to_f32<T>(k_shared[2 * i]), b = to_f32<T>(k_shared[2 * i + 1]);
+        const float a = to_f32<T>(k_shared[first * i]), b = to_f32<T>(k_shared[first * i + apart]);
         const float c = c_row[i], s = s_row[i];
-        T* dst = cache + kv_offset_sized(kv, page, 0, h, in_page) + plain + 2 * i;
+        T* dst = cache + kv_offset_sized(kv, page, 0, h, in_page) + plain + first * i;
         dst[0] = from_f32<T>(a * c - b * s);
-        dst[1] = from_f32<T>(b * c + a * s);
+        dst[apart] = from_f32<T>(b * c + a * s);
     }
     // values: the cache's rows may be wider than the values (padded to the keys' size); the rest is zero
     for (int e = threadIdx.x; e < n_heads * DV; e += blockDim.x) {
@@ -123,7 +126,8 @@ THN_API int thn_latent_assemble(void* q_out, const void* q_src, long long q_stri
                                 long long shared_stride, const void* up, const float* cos_tab, const float* sin_tab,
                                 int table_len, const int* row_slot, const int* row_pos, void* kv_base,
                                 const int* block_table, int bt_stride, int page_size, int n_rows, int n_heads, int plain,
-                                int rot, int value_dim, int value_src, int dtype, int* err, cudaStream_t stream) {
+                                int rot, int interleaved, int value_dim, int value_src, int dtype, int* err,
+                                cudaStream_t stream) {
     THN_CHECK_ARG(n_rows >= 0 && n_heads > 0 && plain >= 0 && rot >= 0 && rot % 2 == 0 && plain + rot > 0 && value_src > 0 &&
                       value_dim >= value_src && page_size > 0,
                   "latent_assemble: bad sizes");
@@ -135,11 +139,11 @@ THN_API int thn_latent_assemble(void* q_out, const void* q_src, long long q_stri
     if (dtype == THN_F32)
         thn_launch(latent_assemble_kernel<float>, n_rows, 256, 0, stream, (float*)q_out, (const float*)q_src, q_stride,
                    (const float*)shared_src, shared_stride, (const float*)up, cos_tab, sin_tab, table_len, row_slot, row_pos,
-                   kv, n_heads, plain, rot, value_src, err);
+                   kv, n_heads, plain, rot, interleaved, value_src, err);
     else if (dtype == THN_BF16)
         thn_launch(latent_assemble_kernel<__nv_bfloat16>, n_rows, 256, 0, stream, (__nv_bfloat16*)q_out,
                    (const __nv_bfloat16*)q_src, q_stride, (const __nv_bfloat16*)shared_src, shared_stride,
-                   (const __nv_bfloat16*)up, cos_tab, sin_tab, table_len, row_slot, row_pos, kv, n_heads, plain, rot, value_src, err);
+                   (const __nv_bfloat16*)up, cos_tab, sin_tab, table_len, row_slot, row_pos, kv, n_heads, plain, rot, interleaved, value_src, err);
     else
         THN_CHECK_ARG(false, "latent_assemble: unknown dtype %d", dtype);
     return thn_launch_status("latent_assemble");

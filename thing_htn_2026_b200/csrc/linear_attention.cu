@@ -12,6 +12,8 @@
 // silu_inputs they pass silu first.  Everything after the load is float32: the state, the decay
 // with its softplus and exponential, the sums.
 //
+// Other mixers use the same recurrence with other decays and read-outs: linear_attention.cuh.
+//
 // Two kernels.  linear_attention_prepare does what is the same for every column, once per entry:
 // silu of q, k and v where asked, the decay with its softplus and exponential, all to float32 rows
 // [row][head][k | q | (decay) | v], the key parts filled up with zeros to a multiple of 32 and the
@@ -26,12 +28,12 @@
 // result depends on its sequence's own tokens only, in an order fixed by the sizes.
 #include <math.h>
 
-#include "common.cuh"
+#include "linear_attention.cuh"
 
 namespace {
 
-constexpr int kLanes = 8;
-constexpr int kColumns = 16;                  // columns of S per block
+constexpr int kLanes = kRecurrenceLanes;
+constexpr int kColumns = kRecurrenceColumns;  // columns of S per block
 constexpr int kThreads = kLanes * kColumns;   // 128
 // tokens per stage: fewer for long keys, so that a thread's share of a stage stays in registers
 constexpr int stage_tokens(int per) { return per <= 16 ? 16 : per <= 32 ? 8 : 4; }
@@ -88,17 +90,19 @@ __global__ void linear_attention_prepare_kernel(float* __restrict__ prepared, co
 }
 
 // PER: key channels per lane (a multiple of 4); KP = 8 * PER: the padded key size.
-// FETCH: 16-byte pieces per thread and stage, ceil(stage tokens * (parts * KP + 16) / 4 / 128).
-template <int PER, int MODE, int FETCH>
+// FETCH: 16-byte pieces per thread and stage, ceil(stage tokens * (parts * KP + 16 + tail) / 4 / 128).
+template <int PER, int KIND, int FETCH>
 __global__ void __launch_bounds__(kThreads) linear_attention_kernel(
-    float* __restrict__ o, float* __restrict__ state, const float* __restrict__ prepared, int vp,
-    const float* __restrict__ decay, const int* __restrict__ cu_seqlens, const int* __restrict__ slots, int n_heads,
-    int key_dim, int value_dim, float q_scale) {
+    float* __restrict__ o, float* __restrict__ state, const float* __restrict__ keys, long long key_stride, int heads_per_unit,
+    const float* __restrict__ values, long long value_stride, const float* __restrict__ per_head,
+    const int* __restrict__ cu_seqlens, const int* __restrict__ slots, int n_heads, int key_dim, int value_dim, int vp,
+    float q_scale) {
     pdl_launch_dependents();
     pdl_wait();
     constexpr int KP = kLanes * PER, kStage = stage_tokens(PER);
-    constexpr int PARTS = MODE == 1 ? 3 : 2;            // k, q (and the decay) per token
-    constexpr int ROW = PARTS * KP + kColumns;          // floats of one staged token
+    constexpr int PARTS = KIND == kChannelDecay || KIND == kBonusRead ? 3 : 2;     // k, q (and the decay) per token
+    constexpr int TAIL = KIND >= kBonusRead ? kRecurrenceTail : 0;
+    constexpr int ROW = PARTS * KP + kColumns + TAIL;   // floats of one staged token
     constexpr int PIECES = ROW / 4;
     extern __shared__ __align__(16) float stage_mem[];  // [2][kStage][ROW]
     const int seq = blockIdx.z, head = blockIdx.y;
@@ -110,7 +114,7 @@ __global__ void __launch_bounds__(kThreads) linear_attention_kernel(
     const int row0 = cu_seqlens[seq], row1 = cu_seqlens[seq + 1];
     const int slot = slots[seq];
     float* S = state + (((size_t)slot * n_heads + head) * value_dim + col) * key_dim;
-    const size_t per_head = (size_t)PARTS * KP + vp;
+    const int unit = head / heads_per_unit, n_units = n_heads / heads_per_unit;
 
     float s[PER];
 #pragma unroll
@@ -118,7 +122,7 @@ __global__ void __launch_bounds__(kThreads) linear_attention_kernel(
         const int d = (i / 4) * 32 + lane * 4 + (i & 3);
         s[i] = d < key_dim ? S[d] : 0.f;
     }
-    const float constant = MODE == 0 ? decay[head] : 1.f;
+    const float own = per_head != nullptr ? per_head[head] : 0.f;      // the constant decay, or the skip's factor
 
     float4 fetched[FETCH];
     auto fetch = [&](int first_row) {
@@ -128,8 +132,14 @@ __global__ void __launch_bounds__(kThreads) linear_attention_kernel(
             const int piece = threadIdx.x + j * kThreads;
             const int t = piece / PIECES, c = (piece - t * PIECES) * 4;
             if (t < n) {
-                const float* src = prepared + ((size_t)(first_row + t) * n_heads + head) * per_head;
-                fetched[j] = *reinterpret_cast<const float4*>(c < PARTS * KP ? src + c : src + c + col0);
+                const float* src;
+                if (c < PARTS * KP) {
+                    src = keys + ((size_t)(first_row + t) * n_units + unit) * key_stride + c;
+                } else {
+                    src = values + ((size_t)(first_row + t) * n_heads + head) * value_stride + (c - PARTS * KP);
+                    src += TAIL != 0 && c >= PARTS * KP + kColumns ? vp - kColumns : col0;
+                }
+                fetched[j] = *reinterpret_cast<const float4*>(src);
             }
         }
     };
@@ -161,24 +171,36 @@ __global__ void __launch_bounds__(kThreads) linear_attention_kernel(
 #pragma unroll 2
         for (int t = 0; t < n; ++t) {
             const float* tok = src + t * ROW;
-            const float v = tok[v_at];
+            const float shown = tok[v_at];
+            float v = shown, decay = own, bonus = 0.f;
+            if (KIND == kBonusRead) bonus = tok[PARTS * KP + kColumns];
+            if (KIND == kSteppedDecay) {
+                decay = tok[PARTS * KP + kColumns];
+                v = shown * tok[PARTS * KP + kColumns + 1];
+            }
             float part = 0.f;
 #pragma unroll
             for (int i = 0; i < PER; i += 4) {
                 const int d = (i / 4) * 32 + lane * 4;
                 const float4 k = *reinterpret_cast<const float4*>(tok + d);
                 const float4 q = *reinterpret_cast<const float4*>(tok + KP + d);
-                float4 a = make_float4(constant, constant, constant, constant);
-                if (MODE == 1) a = *reinterpret_cast<const float4*>(tok + 2 * KP + d);
+                float4 a = make_float4(decay, decay, decay, decay);
+                if (PARTS == 3) a = *reinterpret_cast<const float4*>(tok + 2 * KP + d);
+                if (KIND == kBonusRead) part += s[i] * q.x + s[i + 1] * q.y + s[i + 2] * q.z + s[i + 3] * q.w;
                 s[i] = a.x * s[i] + k.x * v;
                 s[i + 1] = a.y * s[i + 1] + k.y * v;
                 s[i + 2] = a.z * s[i + 2] + k.z * v;
                 s[i + 3] = a.w * s[i + 3] + k.w * v;
-                part += s[i] * q.x + s[i + 1] * q.y + s[i + 2] * q.z + s[i + 3] * q.w;
+                if (KIND != kBonusRead) part += s[i] * q.x + s[i + 1] * q.y + s[i + 2] * q.z + s[i + 3] * q.w;
             }
 #pragma unroll
             for (int off = kLanes / 2; off > 0; off >>= 1) part += __shfl_xor_sync(0xffffffffu, part, off);
-            if (lane == 0 && live) o[((size_t)(first + t) * n_heads + head) * value_dim + col] = part * q_scale;
+            if (lane == 0 && live) {
+                float y = part * q_scale;
+                if (KIND == kBonusRead) y += bonus * shown;
+                if (KIND == kSteppedDecay) y += own * shown;
+                o[((size_t)(first + t) * n_heads + head) * value_dim + col] = y;
+            }
         }
         if (more) publish(buf ^ 1, min(kStage, row1 - first - kStage));
         __syncthreads();
@@ -192,17 +214,29 @@ __global__ void __launch_bounds__(kThreads) linear_attention_kernel(
     }
 }
 
-template <int PER, int MODE>
-void launch_one(float* o, float* state, const float* prepared, int vp, const float* decay, const int* cu_seqlens,
-                const int* slots, int n_seqs, int n_heads, int key_dim, int value_dim, float q_scale, cudaStream_t stream) {
-    constexpr int KP = kLanes * PER, ROW = (MODE == 1 ? 3 : 2) * KP + kColumns, kStage = stage_tokens(PER);
+template <int PER, int KIND>
+void launch_one(const RecurrenceArgs& a, cudaStream_t stream) {
+    constexpr int KP = kLanes * PER, kStage = stage_tokens(PER);
+    constexpr int ROW = (KIND == kChannelDecay || KIND == kBonusRead ? 3 : 2) * KP + kColumns + (KIND >= kBonusRead ? kRecurrenceTail : 0);
     constexpr int FETCH = (kStage * ROW / 4 + kThreads - 1) / kThreads;
     const size_t smem = 2 * (size_t)kStage * ROW * sizeof(float);
-    const dim3 grid((value_dim + kColumns - 1) / kColumns, n_heads, n_seqs);
-    auto kernel = linear_attention_kernel<PER, MODE, FETCH>;
+    const dim3 grid((a.value_dim + kColumns - 1) / kColumns, a.n_heads, a.n_seqs);
+    auto kernel = linear_attention_kernel<PER, KIND, FETCH>;
     if (smem > 48 * 1024) cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-    thn_launch_ordered(kernel, grid, kThreads, smem, stream, o, state, prepared, vp, decay, cu_seqlens, slots, n_heads, key_dim,
-                       value_dim, q_scale);
+    thn_launch_ordered(kernel, grid, kThreads, smem, stream, a.o, a.state, a.keys, a.key_stride, a.n_heads / a.key_units, a.values,
+                       a.value_stride, a.per_head, a.cu_seqlens, a.slots, a.n_heads, a.key_dim, a.value_dim,
+                       padded_values(a.value_dim), a.q_scale);
+}
+
+template <int KIND>
+void launch_kind(const RecurrenceArgs& a, cudaStream_t stream) {
+    switch (recurrence_per_lane(a.key_dim)) {
+        case 4: return launch_one<4, KIND>(a, stream);
+        case 8: return launch_one<8, KIND>(a, stream);
+        case 16: return launch_one<16, KIND>(a, stream);
+        case 32: return launch_one<32, KIND>(a, stream);
+        default: return launch_one<64, KIND>(a, stream);
+    }
 }
 
 template <typename T>
@@ -210,37 +244,38 @@ int launch(float* o, float* state, float* prepared, const void* proj, int proj_w
            const float* decay, const float* gate, int gate_width, const float* gate_bias, float inv_tau,
            const int* cu_seqlens, const int* slots, int n_rows, int n_seqs, int n_heads, int key_dim, int value_dim,
            float q_scale, int mode, int silu_inputs, cudaStream_t stream) {
-    const int per = (key_dim + 31) / 32 * 4;          // runs of four channels per lane
-    const int per_t = per <= 4 ? 4 : per <= 8 ? 8 : per <= 16 ? 16 : per <= 32 ? 32 : 64;
-    const int kp = kLanes * per_t, vp = (value_dim + kColumns - 1) / kColumns * kColumns, parts = mode == 1 ? 3 : 2;
-    const long long n = (long long)n_rows * n_heads * (parts * kp + vp);
+    const int kp = padded_keys(key_dim), vp = padded_values(value_dim), parts = key_parts(mode), per_head = parts * kp + vp;
+    const long long n = (long long)n_rows * n_heads * per_head;
     thn_launch(linear_attention_prepare_kernel<T>, (unsigned)((n + 255) / 256), 256, 0, stream, prepared, (const T*)proj,
                proj_width, q_offset, k_offset, v_offset, gate, gate_width, gate_bias, inv_tau, n, n_heads, key_dim, value_dim, kp,
                vp, parts, silu_inputs);
-#define THN_LA_PER(P)                                                                                                       \
-    do {                                                                                                                    \
-        if (mode == 0) launch_one<P, 0>(o, state, prepared, vp, decay, cu_seqlens, slots, n_seqs, n_heads, key_dim, value_dim, \
-                                        q_scale, stream);                                                                   \
-        else launch_one<P, 1>(o, state, prepared, vp, decay, cu_seqlens, slots, n_seqs, n_heads, key_dim, value_dim, q_scale, \
-                              stream);                                                                                      \
-    } while (0)
-    if (per_t == 4) THN_LA_PER(4);
-    else if (per_t == 8) THN_LA_PER(8);
-    else if (per_t == 16) THN_LA_PER(16);
-    else if (per_t == 32) THN_LA_PER(32);
-    else THN_LA_PER(64);
-#undef THN_LA_PER
-    return thn_launch_status("linear_attention");
+    return launch_recurrence(mode, RecurrenceArgs{o, state, prepared, per_head, n_heads, prepared + parts * kp, per_head, decay,
+                                                  cu_seqlens, slots, n_seqs, n_heads, key_dim, value_dim, q_scale},
+                             stream);
 }
 
 }  // namespace
 
+int launch_recurrence(int kind, const RecurrenceArgs& args, cudaStream_t stream) {
+    THN_CHECK_ARG(args.key_units > 0 && args.n_heads % args.key_units == 0, "recurrence: %d heads over %d units of keys",
+                  args.n_heads, args.key_units);
+    THN_UNSUPPORTED_IF(args.key_dim > 512, "recurrence: keys of %d, at most 512", args.key_dim);
+    THN_UNSUPPORTED_IF(args.n_heads > 65535 || args.n_seqs > 65535, "recurrence: %d heads, %d sequences", args.n_heads, args.n_seqs);
+    THN_CHECK_ARG((((uintptr_t)args.keys | (uintptr_t)args.values) & 15) == 0 && args.key_stride % 4 == 0 && args.value_stride % 4 == 0,
+                  "recurrence: prepared rows are not 16-byte aligned");
+    switch (kind) {
+        case kConstantDecay: launch_kind<kConstantDecay>(args, stream); break;
+        case kChannelDecay: launch_kind<kChannelDecay>(args, stream); break;
+        case kBonusRead: launch_kind<kBonusRead>(args, stream); break;
+        case kSteppedDecay: launch_kind<kSteppedDecay>(args, stream); break;
+        default: THN_CHECK_ARG(false, "recurrence: unknown kind %d", kind);
+    }
+    return thn_launch_status("recurrence");
+}
+
 // Floats of the scratch that thn_linear_attention needs for a step of n_rows rows.
 THN_API long long thn_linear_attention_scratch_floats(int n_rows, int n_heads, int key_dim, int value_dim, int mode) {
-    const int per = (key_dim + 31) / 32 * 4;
-    const int per_t = per <= 4 ? 4 : per <= 8 ? 8 : per <= 16 ? 16 : per <= 32 ? 32 : 64;
-    const long long kp = kLanes * per_t, vp = (value_dim + kColumns - 1) / kColumns * kColumns;
-    return (long long)n_rows * n_heads * ((mode == 1 ? 3 : 2) * kp + vp);
+    return (long long)n_rows * n_heads * ((mode == 1 ? 3 : 2) * (long long)padded_keys(key_dim) + padded_values(value_dim));
 }
 
 // o float32 [rows, heads, value_dim]; state float32 [slots, heads, value_dim, key_dim], read and

@@ -1,7 +1,9 @@
 // Routing of a mixture of experts, and the experts' activation with the routing weights.
 //
 //   moe_route   per row: scores s = softmax(z) over all experts (scoring 0) or s = logistic(z),
-//               each expert by itself (scoring 1); the experts form `groups` equal
+//               each expert by itself (scoring 1), or none over all experts: the choice is made on the
+//               logits and the weights are the softmax over the chosen logits alone (scoring 2, one
+//               group only); the experts form `groups` equal
 //               groups of neighbours, a group's score is its largest s, and only experts of the
 //               `keep` best groups can be chosen; the `top` allowed experts with the largest s
 //               are chosen (the lower index wins a tie); a chosen expert's weight is s * scale,
@@ -21,6 +23,8 @@
 //               A row holds [gates of all columns | ups of all columns]; the columns are
 //               [experts * ff | shared_ff].  The shared expert sees the token itself, has a limit
 //               of its own, and its columns are multiplied by logistic(gate logit of the row).
+//               What is added to u (1 above) is a parameter, and limits may be infinite: with slope 1, no
+//               limit and nothing added it is the plain silu(gate) * up.
 //               With weight_output the routing weight multiplies the expert's activation instead
 //               (the expert sees the token itself and its output is weighted).
 #include <math.h>
@@ -61,9 +65,9 @@ __global__ void __launch_bounds__(kRouteWarps * 32) moe_route_kernel(
     const float* zr = z + (size_t)row * z_stride;
     const int per = n_experts / n_groups;
 
-    if (scoring == 1 && keep >= n_groups) {
-        // Logistic scores of experts that are all eligible: the order of the scores is the order
-        // of the logits, and the logits do not saturate, so the choice is made on them.
+    if (scoring == 2 || (scoring == 1 && keep >= n_groups)) {
+        // Experts that are all eligible, with scores whose order is the order of the logits: the
+        // logits do not saturate, so the choice is made on them.
         for (int e = lane; e < n_experts; e += 32) {
             s[e] = zr[e];
             dense[(size_t)row * n_experts + e] = 0.f;
@@ -77,17 +81,29 @@ __global__ void __launch_bounds__(kRouteWarps * 32) moe_route_kernel(
             __syncwarp();
             if (lane == 0) {
                 if (b.index < n_experts) {
-                    const float w = scale / (1.0f + expf(-b.value));
+                    // (scoring 2: the logit itself, until all are chosen)
+                    const float w = scoring == 2 ? b.value : scale / (1.0f + expf(-b.value));
                     dense[(size_t)row * n_experts + b.index] = w;
                     chosen[(size_t)row * top + pick] = b.index;
                     chosen_weight[(size_t)row * top + pick] = w;
                     s[b.index] = -INFINITY;       // taken
                 } else {                      // no logit compares (not a number): an index that exists, no weight
                     chosen[(size_t)row * top + pick] = pick;
-                    chosen_weight[(size_t)row * top + pick] = 0.f;
+                    chosen_weight[(size_t)row * top + pick] = scoring == 2 ? -INFINITY : 0.f;
                 }
             }
             __syncwarp();
+        }
+        if (scoring == 2 && lane == 0) {
+            // softmax over the chosen logits; the first one chosen is the largest
+            float* w = chosen_weight + (size_t)row * top;
+            const float most = w[0];
+            float sum = 0.f;
+            for (int pick = 0; pick < top; ++pick) sum += expf(w[pick] - most);
+            for (int pick = 0; pick < top; ++pick) {
+                w[pick] = scale * expf(w[pick] - most) / sum;
+                dense[(size_t)row * n_experts + chosen[(size_t)row * top + pick]] = w[pick];
+            }
         }
         return;
     }
@@ -220,7 +236,7 @@ template <typename T>
 __global__ void routed_clamped_glu_kernel(T* __restrict__ out, const T* __restrict__ gu, const float* __restrict__ dense,
                                           const float* __restrict__ shared_logit, long long logit_stride, long long n,
                                           int width, int n_experts, int ff, float limit, float shared_limit, float alpha,
-                                          int weight_output) {
+                                          float up_shift, int weight_output) {
     pdl_launch_dependents();
     pdl_wait();
     const long long e = (long long)blockIdx.x * blockDim.x + threadIdx.x;
@@ -239,7 +255,7 @@ __global__ void routed_clamped_glu_kernel(T* __restrict__ out, const T* __restri
     const T* src = gu + row * 2 * width;
     const float g = fminf(w * to_f32<T>(src[c]), lim);
     const float u = fminf(fmaxf(w * to_f32<T>(src[width + c]), -lim), lim);
-    out[e] = from_f32<T>(g / (1.0f + expf(-alpha * g)) * (u + 1.0f) * after);
+    out[e] = from_f32<T>(g / (1.0f + expf(-alpha * g)) * (u + up_shift) * after);
 }
 
 // The same, eight bfloat16 columns per thread (16-byte accesses), one row per blockIdx.y: for
@@ -247,7 +263,7 @@ __global__ void routed_clamped_glu_kernel(T* __restrict__ out, const T* __restri
 __global__ void routed_clamped_glu_bf16_vec_kernel(__nv_bfloat16* __restrict__ out, const __nv_bfloat16* __restrict__ gu,
                                                    const float* __restrict__ dense, const float* __restrict__ shared_logit,
                                                    long long logit_stride, int width, int n_experts, int ff, float limit,
-                                                   float shared_limit, float alpha, int weight_output) {
+                                                   float shared_limit, float alpha, float up_shift, int weight_output) {
     pdl_launch_dependents();
     pdl_wait();
     const int c = (blockIdx.x * blockDim.x + threadIdx.x) * 8;
@@ -273,8 +289,8 @@ __global__ void routed_clamped_glu_bf16_vec_kernel(__nv_bfloat16* __restrict__ o
             const float2 g = __bfloat1622float2(g2[j]), u = __bfloat1622float2(u2[j]);
             const float g0 = fminf(w * g.x, lim), g1 = fminf(w * g.y, lim);
             const float u0 = fminf(fmaxf(w * u.x, -lim), lim), u1 = fminf(fmaxf(w * u.y, -lim), lim);
-            ob[j] = __floats2bfloat162_rn(g0 / (1.0f + expf(-alpha * g0)) * (u0 + 1.0f) * after,
-                                          g1 / (1.0f + expf(-alpha * g1)) * (u1 + 1.0f) * after);
+            ob[j] = __floats2bfloat162_rn(g0 / (1.0f + expf(-alpha * g0)) * (u0 + up_shift) * after,
+                                          g1 / (1.0f + expf(-alpha * g1)) * (u1 + up_shift) * after);
         }
     }
     *reinterpret_cast<uint4*>(out + row * width + c) = packed;
@@ -289,7 +305,8 @@ THN_API int thn_moe_route(float* dense, int* chosen, float* chosen_weight, const
                           float renorm_eps, cudaStream_t stream) {
     THN_CHECK_ARG(n_rows >= 0 && n_experts > 0 && n_groups > 0 && n_experts % n_groups == 0,
                   "moe_route: %d experts in %d groups", n_experts, n_groups);
-    THN_CHECK_ARG(scoring == 0 || scoring == 1, "moe_route: scoring %d (0: softmax, 1: logistic)", scoring);
+    THN_CHECK_ARG(scoring >= 0 && scoring <= 2, "moe_route: scoring %d (0: softmax, 1: logistic, 2: softmax over the chosen)", scoring);
+    THN_CHECK_ARG(scoring != 2 || keep == n_groups, "moe_route: a softmax over the chosen leaves no group out");
     THN_CHECK_ARG(!renormalise || (scoring == 0 && scale != 0.f), "moe_route: weights are renormalised with softmax scores only");
     THN_CHECK_ARG(keep > 0 && keep <= n_groups && top > 0 && top <= keep * (n_experts / n_groups),
                   "moe_route: top %d of the experts of %d groups out of %d", top, keep, n_groups);
@@ -335,7 +352,8 @@ THN_API int thn_routed_gelu(void* out, const void* u, const float* dense, const 
 // rows' gate logits of the shared expert, logit_stride apart (null: no gate).
 THN_API int thn_routed_clamped_glu(void* out, const void* gu, const float* dense, const float* shared_logit,
                                    long long logit_stride, int n_rows, int n_experts, int ff, int shared_ff, float limit,
-                                   float shared_limit, float alpha, int weight_output, int dtype, cudaStream_t stream) {
+                                   float shared_limit, float alpha, float up_shift, int weight_output, int dtype,
+                                   cudaStream_t stream) {
     THN_CHECK_ARG(n_rows >= 0 && n_experts >= 0 && ff >= 0 && shared_ff >= 0 && n_experts * ff + shared_ff > 0,
                   "routed_clamped_glu: bad sizes");
     THN_CHECK_ARG((n_experts * ff == 0 || limit > 0.f) && (shared_ff == 0 || shared_limit > 0.f),
@@ -348,16 +366,16 @@ THN_API int thn_routed_clamped_glu(void* out, const void* gu, const float* dense
         ((((uintptr_t)out) | ((uintptr_t)gu)) & 15) == 0) {
         thn_launch(routed_clamped_glu_bf16_vec_kernel, dim3((width / 8 + 127) / 128, n_rows), 128, 0, stream,
                    (__nv_bfloat16*)out, (const __nv_bfloat16*)gu, dense, shared_logit, logit_stride, width, n_experts, ff,
-                   limit, shared_limit, alpha, weight_output);
+                   limit, shared_limit, alpha, up_shift, weight_output);
         return thn_launch_status("routed_clamped_glu");
     }
     if (dtype == THN_F32)
         thn_launch(routed_clamped_glu_kernel<float>, blocks, 256, 0, stream, (float*)out, (const float*)gu, dense,
-                   shared_logit, logit_stride, n, width, n_experts, ff, limit, shared_limit, alpha, weight_output);
+                   shared_logit, logit_stride, n, width, n_experts, ff, limit, shared_limit, alpha, up_shift, weight_output);
     else if (dtype == THN_BF16)
         thn_launch(routed_clamped_glu_kernel<__nv_bfloat16>, blocks, 256, 0, stream, (__nv_bfloat16*)out,
                    (const __nv_bfloat16*)gu, dense, shared_logit, logit_stride, n, width, n_experts, ff, limit, shared_limit,
-                   alpha, weight_output);
+                   alpha, up_shift, weight_output);
     else
         THN_CHECK_ARG(false, "routed_clamped_glu: unknown dtype %d", dtype);
     return thn_launch_status("routed_clamped_glu");

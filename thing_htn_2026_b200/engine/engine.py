@@ -98,6 +98,10 @@ class Engine:
             for t in ids:
                 if not 0 <= int(t) < vocab:
                     raise ValueError(f"sequence {i}: token id {t} is outside the vocabulary [0, {vocab})")
+            # (the last new token is returned, not fed back)
+            if self.model.position_limit is not None and len(ids) + limits[i] - 1 > self.model.position_limit:
+                raise ValueError(f"sequence {i}: {len(ids)} tokens and {limits[i]} new ones do not fit the model's "
+                                 f"{self.model.position_limit} positions")
         return [Request(list(ids), limits[i], temps[i], int(seed), i, tuple(stop_token_ids or ()))
                 for i, ids in enumerate(input_ids)]
 

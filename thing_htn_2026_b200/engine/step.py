@@ -38,6 +38,8 @@ class StepRunner:
         self.device = model.device
         self.err = ops.new_error_word(self.device)
         model.ensure_positions(cache.max_pages_per_seq * cache.page_size)
+        for name, (shape, dtype) in model.sequence_states().items():     # before any step is captured as a graph
+            cache.sequence_state(name, shape, dtype)
         # Host-to-device uploads go through a small ring of pinned buffers; a buffer is reused
         # only after the copy that read it has finished.
         self._staging = [[None, None] for _ in range(4)]     # [pinned int32 tensor, event]
@@ -83,7 +85,7 @@ class StepRunner:
     def step(self, entries: Sequence[StepEntry], check: bool = True) -> torch.Tensor:
         """Runs the entries' tokens; returns float32 logits ``[wanted, vocab]`` in the order
         of the entries and of their ``want``.  Raises CacheFull before touching anything if
-        the cache cannot take the tokens."""
+        the cache cannot take the tokens, and ValueError if a sequence outgrows the model's positions."""
         entries = [e for e in entries]
         slots = [e.slot for e in entries]
         counts = [len(e.tokens) for e in entries]
@@ -99,6 +101,10 @@ class StepRunner:
                 if not 0 <= w < len(e.tokens):
                     raise ValueError(f"slot {e.slot}: wanted place {w} is outside its {len(e.tokens)} tokens")
                 want_rows.append(start + w)
+        limit = self.model.position_limit
+        for slot, count in zip(slots, counts):
+            if limit is not None and self.cache.length(slot) + count > limit:
+                raise ValueError(f"slot {slot}: {self.cache.length(slot) + count} tokens, the model has {limit} positions")
         self.cache.prepare(slots, counts)
         held = [self.cache.length(slot) for slot in slots]
 

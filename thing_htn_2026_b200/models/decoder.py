@@ -69,6 +69,15 @@ class DecoderModel:
                 needs[entry.cache] = self.layers[entry.layer].cache_need()
         return needs
 
+    def sequence_states(self) -> Dict[str, tuple]:
+        """Named per-sequence state that parts outside the cache entries keep: name -> (shape, dtype)."""
+        return self.embedding.sequence_states() if hasattr(self.embedding, "sequence_states") else {}
+
+    @property
+    def position_limit(self) -> Optional[int]:
+        """The most positions a sequence can have, where a table of the model sets it (None: no limit)."""
+        return getattr(self.embedding, "position_limit", None)
+
     def ensure_positions(self, n_positions: int) -> None:
         for part in self.runtime.shared.values():
             if hasattr(part, "ensure"):
@@ -87,7 +96,7 @@ class DecoderModel:
     def hidden(self, tokens: torch.Tensor, ctx: StepContext):
         """All scheduled layers over the step's rows; returns the residual stream and the
         last branch output that has not been added yet."""
-        h = self.embedding.forward(tokens, ctx.err, ctx.rows)
+        h = self.embedding.forward(tokens, ctx.err, ctx.rows, ctx.cache)
         d: Optional[torch.Tensor] = None
         for entry in self.plan.schedule:
             h, d = self.layers[entry.layer].forward(h, d, ctx, entry)

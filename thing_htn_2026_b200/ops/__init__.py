@@ -77,15 +77,32 @@ _SIGNATURES = {
     "thn_add_bias_f32": [c_void_p, c_void_p, c_int, c_int, c_float, c_void_p],
     "thn_gather_rows_scaled": [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_float, c_void_p, c_void_p, c_int,
                                c_void_p, c_void_p],
+    "thn_embed_rows": [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_float, c_void_p, c_int, c_longlong, c_longlong,
+                       c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_void_p, c_void_p],
+    "thn_squared_relu": [c_void_p, c_void_p, c_longlong, c_int, c_void_p],
+    "thn_token_shift": [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int,
+                        c_int, c_int, c_void_p],
+    "thn_tanh_rows": [c_void_p, c_void_p, c_longlong, c_int, c_void_p],
+    "thn_wkv": [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
+                c_int, c_int, c_int, c_int, c_int, c_void_p],
+    "thn_wkv_decode": [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p,
+                       c_void_p, c_void_p, c_float, c_void_p, c_int, c_int, c_int, c_int, c_void_p],
+    "thn_state_space": [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
+                        c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int,
+                        c_int, c_int, c_int, c_int, c_void_p],
+    "thn_state_space_decode": [c_void_p, c_void_p, c_void_p, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
+                               c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int,
+                               c_void_p],
+    "thn_gated_group_norm": [c_void_p, c_void_p, c_void_p, c_longlong, c_void_p, c_float, c_int, c_int, c_int, c_int, c_void_p],
     "thn_scale_f32": [c_void_p, c_longlong, c_float, c_void_p],
     "thn_polynorm": [c_void_p, c_void_p, c_void_p, c_int, c_int, c_float, c_int, c_void_p],
     "thn_routed_clamped_glu": [c_void_p, c_void_p, c_void_p, c_void_p, c_longlong, c_int, c_int, c_int, c_int, c_float,
-                               c_float, c_float, c_int, c_int, c_void_p],
-    "thn_logistic_gate": [c_void_p, c_void_p, c_void_p, c_longlong, c_int, c_int, c_int, c_void_p],
+                               c_float, c_float, c_float, c_int, c_int, c_void_p],
+    "thn_logistic_gate": [c_void_p, c_void_p, c_void_p, c_longlong, c_int, c_int, c_int, c_int, c_void_p],
     "thn_latent_norm": [c_void_p, c_void_p, c_longlong, c_void_p, c_float, c_int, c_int, c_int, c_void_p],
     "thn_latent_assemble": [c_void_p, c_void_p, c_longlong, c_void_p, c_longlong, c_void_p, c_void_p, c_void_p, c_int,
                             c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int,
-                            c_int, c_void_p, c_void_p],
+                            c_int, c_int, c_void_p, c_void_p],
     "thn_mlstm_columns_per_block": [],
     "thn_mlstm_gates": [c_void_p, c_void_p, c_void_p, c_void_p, c_float, c_int, c_int, c_void_p],
     "thn_mlstm_recurrence": [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_float, c_int,
@@ -172,6 +189,10 @@ def lib():
         loaded.thn_attention_decode_scratch_floats.restype = c_longlong
         loaded.thn_linear_attention_scratch_floats.argtypes = [c_int, c_int, c_int, c_int, c_int]
         loaded.thn_linear_attention_scratch_floats.restype = c_longlong
+        loaded.thn_wkv_scratch_floats.argtypes = [c_int, c_int, c_int]
+        loaded.thn_wkv_scratch_floats.restype = c_longlong
+        loaded.thn_state_space_scratch_floats.argtypes = [c_int, c_int, c_int, c_int, c_int]
+        loaded.thn_state_space_scratch_floats.restype = c_longlong
         _lib = loaded
     return _lib
 
@@ -338,6 +359,61 @@ def gather_rows_scaled(table: torch.Tensor, index: torch.Tensor, scale: float,
     return out
 
 
+@dataclass
+class PairTable:
+    """Rows for pairs of neighbouring tokens: ``table`` [buckets + 1, width]; the pair (before, token)
+    takes row ``(before * mul_before + token * mul_token) mod buckets``, a sequence's first token the
+    last row."""
+
+    table: torch.Tensor
+    mul_before: int
+    mul_token: int
+
+    @property
+    def buckets(self) -> int:
+        return self.table.shape[0] - 1
+
+
+def embed_rows(table: torch.Tensor, tokens: torch.Tensor, scale: float, rows: StepRows, seq_lens: torch.Tensor,
+               pairs: Optional[PairTable] = None, previous: Optional[torch.Tensor] = None,
+               positions: Optional[torch.Tensor] = None, err: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """The rows that start a float32 residual stream: ``table[token] * scale``, plus the row of the
+    token's pair with the one before it, plus ``positions[pos]`` (learned position vectors; a position
+    beyond the table sets ERR_POSITION_RANGE).  The token before the first one that a sequence brings
+    comes from ``previous`` (int32 [slots]), where the step's last token is left; ``seq_lens`` holds the
+    tokens each slot held before the step."""
+    _need(table, "embed_rows table")
+    _need(tokens, "embed_rows tokens", torch.int32)
+    _need(seq_lens, "embed_rows seq_lens", torch.int32)
+    width = table.shape[1]
+    if tokens.shape[0] != rows.n_rows:
+        raise KernelError(f"embed_rows: {tokens.shape[0]} tokens for a step of {rows.n_rows} rows")
+    if pairs is not None:
+        _need(pairs.table, "embed_rows pairs", table.dtype)
+        if previous is None or pairs.table.shape[1] != width or pairs.buckets < 1:
+            raise KernelError(f"embed_rows: pairs {tuple(pairs.table.shape)} for rows of {width}, with the tokens before")
+        _need(previous, "embed_rows previous", torch.int32)
+    if positions is not None:
+        _need(positions, "embed_rows positions", table.dtype)
+        if positions.shape[1] != width:
+            raise KernelError(f"embed_rows: positions {tuple(positions.shape)} for rows of {width}")
+    out = torch.empty((rows.n_rows, width), dtype=torch.float32, device=table.device)
+    _call("thn_embed_rows", _ptr(out), _ptr(table), _ptr(tokens), rows.n_rows, width, table.shape[0], float(scale),
+          _ptr(pairs.table) if pairs else None, pairs.buckets if pairs else 0, int(pairs.mul_before) if pairs else 0,
+          int(pairs.mul_token) if pairs else 0, _ptr(previous) if pairs else None, _ptr(positions),
+          positions.shape[0] if positions is not None else 0, _ptr(rows.row_slot), _ptr(rows.row_pos), _ptr(rows.cu_seqlens),
+          _ptr(seq_lens), rows.n_seqs, _code(table, "embed_rows"), _ptr(err), _stream())
+    return out
+
+
+def squared_relu(z: torch.Tensor) -> torch.Tensor:
+    """max(z, 0)^2, entry by entry."""
+    _need(z, "squared_relu z")
+    out = torch.empty_like(z)
+    _call("thn_squared_relu", _ptr(out), _ptr(z), z.numel(), _code(z, "squared_relu"), _stream())
+    return out
+
+
 def scale_(x: torch.Tensor, scale: float) -> torch.Tensor:
     """x *= scale in place (float32): a constant factor on logits."""
     _need(x, "scale_", torch.float32)
@@ -359,17 +435,18 @@ def polynorm(z: torch.Tensor, coefficients: torch.Tensor, eps: float) -> torch.T
     return out
 
 
-def logistic_gate(a: torch.Tensor, gate: torch.Tensor, gate_offset: int = 0) -> torch.Tensor:
-    """a [rows, width] * logistic(gate[:, gate_offset : gate_offset + width]); the gate may be a
-    slice of a wider projected row."""
+def logistic_gate(a: torch.Tensor, gate: torch.Tensor, gate_offset: int = 0, per: int = 1) -> torch.Tensor:
+    """a [rows, width] * logistic(gate[:, gate_offset + i // per]) at entry i: a gate per entry, or
+    (``per`` neighbours sharing one) a gate per head; the gate may be a slice of a wider projected row."""
     _need(a, "logistic_gate a")
     _need(gate, "logistic_gate gate", a.dtype)
     rows, width = a.shape
-    if gate.shape[0] != rows or gate_offset + width > gate.shape[1]:
-        raise KernelError(f"logistic_gate: shapes a {tuple(a.shape)}, gate {tuple(gate.shape)} from column {gate_offset}")
+    if gate.shape[0] != rows or width % per or gate_offset + width // per > gate.shape[1]:
+        raise KernelError(f"logistic_gate: shapes a {tuple(a.shape)}, gate {tuple(gate.shape)} from column {gate_offset}, "
+                          f"one for {per} entries")
     out = torch.empty_like(a)
     _call("thn_logistic_gate", _ptr(out), _ptr(a), gate.data_ptr() + gate_offset * gate.element_size(), gate.shape[1],
-          rows, width, _code(a, "logistic_gate"), _stream())
+          rows, width, int(per), _code(a, "logistic_gate"), _stream())
     return out
 
 
@@ -692,6 +769,22 @@ def linear(x: torch.Tensor, weight: torch.Tensor, out_dtype: Optional[torch.dtyp
     if out_dtype in (None, torch.bfloat16):
         return torch.nn.functional.linear(x, weight)
     return torch.mm(x, weight.t(), out_dtype=out_dtype)
+
+
+def linear_batched(x: torch.Tensor, weight: torch.Tensor) -> torch.Tensor:
+    """``x [B, M, K]`` and ``weight [B, N, K]`` -> ``[B, M, N]``: several products of one shape on operands
+    of their own.  bfloat16: one batched product of the vendor library; float32: this library's FFMA
+    kernel, one launch each."""
+    _need(x, "linear_batched x")
+    _need(weight, "linear_batched weight", x.dtype)
+    if x.dim() != 3 or weight.dim() != 3 or x.shape[0] != weight.shape[0] or x.shape[2] != weight.shape[2]:
+        raise KernelError(f"linear_batched: shapes x {tuple(x.shape)}, weight {tuple(weight.shape)}")
+    if x.dtype == torch.bfloat16:
+        return torch.bmm(x, weight.transpose(1, 2))
+    out = torch.empty((x.shape[0], x.shape[1], weight.shape[1]), dtype=torch.float32, device=x.device)
+    for b in range(x.shape[0]):
+        _call("thn_gemm_f32", _ptr(out[b]), _ptr(x[b]), _ptr(weight[b]), x.shape[1], weight.shape[1], x.shape[2], _stream())
+    return out
 
 
 # ------------------------------------------------------------------ attention
@@ -1188,7 +1281,7 @@ def latent_assemble(proj: torch.Tensor, q_offset: int, shared_offset: int, up: t
     ``[heads][plain | rot]`` from column ``q_offset`` and one shared key part of ``rot`` entries
     from column ``shared_offset``; ``up`` [rows, heads * plain + heads * value] is the
     up-projection of the normalised latent.  The ``rot`` parts are rotated by the rows' positions
-    (interleaved pairs); the cache gets per head the key ``[plain | rotated shared part]`` and the
+    (pairs as ``rotary.layout`` says); the cache gets per head the key ``[plain | rotated shared part]`` and the
     value.  ``value_dim`` (default: the cache's value size) is the size of a value in ``up``; a
     cache whose values are wider gets zeros behind them.  Returns the queries
     [rows, heads * (plain + rot)]."""
@@ -1202,15 +1295,15 @@ def latent_assemble(proj: torch.Tensor, q_offset: int, shared_offset: int, up: t
         raise KernelError(f"latent_assemble: values of {value_dim} do not fit the cache's {kv.v_dim}")
     if proj.shape[0] != rows.n_rows or tuple(up.shape) != (rows.n_rows, n_heads * (plain + value_dim)):
         raise KernelError(f"latent_assemble: shapes proj {tuple(proj.shape)}, up {tuple(up.shape)} for {rows.n_rows} rows")
-    if rot and (rotary is None or rotary.layout != "interleaved" or rotary.rotary_dim != rot):
-        raise KernelError("latent_assemble: the rotated part needs interleaved tables of its size")
+    if rot and (rotary is None or rotary.rotary_dim != rot):
+        raise KernelError("latent_assemble: the rotated part needs tables of its size")
     q = torch.empty((rows.n_rows, n_heads * (plain + rot)), dtype=proj.dtype, device=proj.device)
     size = proj.element_size()
     _call("thn_latent_assemble", _ptr(q), proj.data_ptr() + q_offset * size, proj.shape[1],
           proj.data_ptr() + shared_offset * size, proj.shape[1], _ptr(up), _ptr(rotary.cos) if rot else None,
           _ptr(rotary.sin) if rot else None, rotary.cos.shape[0] if rot else 0, _ptr(rows.row_slot), _ptr(rows.row_pos),
           _ptr(kv.storage), _ptr(kv.block_table), kv.block_table.shape[1], kv.page_size, rows.n_rows, n_heads, plain, rot,
-          kv.v_dim, value_dim, _code(proj, "latent_assemble"), _ptr(err), _stream())
+          ROTARY_LAYOUTS[rotary.layout] if rot else 0, kv.v_dim, value_dim, _code(proj, "latent_assemble"), _ptr(err), _stream())
     return q
 
 
@@ -1279,14 +1372,15 @@ class Routing:
     chosen_weight: torch.Tensor   # float32 [rows, top]
 
 
-SCORINGS = {"softmax": 0, "logistic": 1}
+SCORINGS = {"softmax": 0, "logistic": 1, "softmax_chosen": 2}
 
 
 def moe_route(logits: torch.Tensor, n_experts: int, n_groups: int, keep: int, top: int, scale: float,
               scoring: str = "softmax", renormalise: Optional[float] = None) -> Routing:
     """Routing weights from float32 router logits (the first ``n_experts`` columns of
     ``logits``): scores by softmax over all experts or (``scoring`` "logistic") the logistic
-    function of each logit, the ``keep`` best of ``n_groups`` groups of neighbours (a group's
+    function of each logit or (``scoring`` "softmax_chosen", one group) a softmax over the chosen
+    logits alone, the ``keep`` best of ``n_groups`` groups of neighbours (a group's
     score is its largest), the ``top`` best allowed experts, weights ``score * scale``.
     ``renormalise`` (a small number, softmax scores only): the chosen experts' scores are divided by
     their sum plus that number first."""
@@ -1305,15 +1399,15 @@ def moe_route(logits: torch.Tensor, n_experts: int, n_groups: int, keep: int, to
 
 def routed_clamped_glu(gu: torch.Tensor, routing: Routing, ff: int, shared_ff: int, limit: float, shared_limit: float,
                        alpha: float, shared_logit: Optional[torch.Tensor] = None, logit_column: int = 0,
-                       weight_at: str = "input") -> torch.Tensor:
-    """Experts ``g * logistic(alpha * g) * (u + 1)`` with ``g = min(w * gate, limit)`` and
+                       weight_at: str = "input", up_shift: float = 1.0) -> torch.Tensor:
+    """Experts ``g * logistic(alpha * g) * (u + up_shift)`` with ``g = min(w * gate, limit)`` and
     ``u = clamp(w * up, -limit, limit)``, ``w`` the routing weight of the column's expert: the
     expert sees the token times its weight, and its projections are linear.  ``gu`` [rows,
     2 * (experts * ff + shared_ff)] holds the gates of all columns, then the ups.  The shared
     expert's columns take ``w = 1`` and ``shared_limit`` and are multiplied by
     ``logistic(shared_logit[:, logit_column])`` (no gate without ``shared_logit``); columns of an
     expert that was not chosen are zero.  ``weight_at`` "output": the expert sees the token itself
-    and ``w`` multiplies its activation instead.  Returns [rows, experts * ff + shared_ff]."""
+    and ``w`` multiplies its activation instead.  Limits may be infinite.  Returns [rows, experts * ff + shared_ff]."""
     if weight_at not in ("input", "output"):
         raise KernelError(f"routed_clamped_glu: weight_at {weight_at!r} is neither 'input' nor 'output'")
     _need(gu, "routed_clamped_glu gu")
@@ -1327,7 +1421,7 @@ def routed_clamped_glu(gu: torch.Tensor, routing: Routing, ff: int, shared_ff: i
         logit_ptr, stride = shared_logit.data_ptr() + 4 * logit_column, shared_logit.shape[1]
     out = torch.empty((rows, width), dtype=gu.dtype, device=gu.device)
     _call("thn_routed_clamped_glu", _ptr(out), _ptr(gu), _ptr(routing.dense), logit_ptr, stride, rows, n_experts, ff,
-          shared_ff, float(limit), float(shared_limit or 1.0), float(alpha), int(weight_at == "output"),
+          shared_ff, float(limit), float(shared_limit or 1.0), float(alpha), float(up_shift), int(weight_at == "output"),
           _code(gu, "routed_clamped_glu"), _stream())
     return out
 
@@ -1514,6 +1608,168 @@ def selective_scan(x: torch.Tensor, dt_pre: torch.Tensor, dt_bias: torch.Tensor,
     return y
 
 
+# ------------------------------------------------------------------ time mixing, state-space duality
+
+
+def token_shift(x: torch.Tensor, mu: torch.Tensor, shift: torch.Tensor, rows: StepRows, seq_lens: torch.Tensor) -> torch.Tensor:
+    """Blends of every row with the row of the token before it: ``out[s] = x + (x' - x) * mu[s]`` for
+    ``mu`` float32 [n, width] -> [n, rows, width].  ``x'`` is the row above, for the first row that a
+    sequence brings what ``shift`` [slots, width] holds (zeros at position 0); the step's last row of
+    each sequence is left there.  ``seq_lens`` holds the tokens each slot held before the step."""
+    _need(x, "token_shift x")
+    _need(mu, "token_shift mu", torch.float32)
+    _need(shift, "token_shift shift", x.dtype)
+    n, width = mu.shape
+    if tuple(x.shape) != (rows.n_rows, width) or shift.shape[1] != width:
+        raise KernelError(f"token_shift: x {tuple(x.shape)}, mu {tuple(mu.shape)}, shift {tuple(shift.shape)}")
+    out = torch.empty((n, rows.n_rows, width), dtype=x.dtype, device=x.device)
+    _call("thn_token_shift", _ptr(out), _ptr(x), _ptr(mu), _ptr(shift), _ptr(rows.row_slot), _ptr(rows.row_pos),
+          _ptr(rows.cu_seqlens), _ptr(seq_lens), rows.n_rows, rows.n_seqs, width, n, _code(x, "token_shift"), _stream())
+    return out
+
+
+def tanh_rows(x: torch.Tensor, dtype: torch.dtype) -> torch.Tensor:
+    """tanh of a float32 tensor, of ``dtype``."""
+    _need(x, "tanh_rows x", torch.float32)
+    out = torch.empty(x.shape, dtype=dtype, device=x.device)
+    _call("thn_tanh_rows", _ptr(out), _ptr(x), x.numel(), DTYPE_CODE[dtype], _stream())
+    return out
+
+
+def _wkv_check(planes: torch.Tensor, w0: torch.Tensor, u: torch.Tensor, state: torch.Tensor, rows: StepRows, n_heads: int,
+               dim: int, what: str) -> None:
+    _need(planes, f"{what} projections")
+    _need(w0, f"{what} w0", torch.float32)
+    _need(u, f"{what} u", torch.float32)
+    _need(state, f"{what} state", torch.float32)
+    if planes.dim() != 3 or planes.shape[0] < 3 or tuple(planes.shape[1:]) != (rows.n_rows, n_heads * dim) \
+            or w0.numel() != n_heads * dim or u.numel() != n_heads * dim or tuple(state.shape[1:]) != (n_heads, dim, dim):
+        raise KernelError(f"{what}: projections {tuple(planes.shape)}, w0 {tuple(w0.shape)}, u {tuple(u.shape)}, state "
+                          f"{tuple(state.shape)} do not fit {n_heads} heads of {dim} over {rows.n_rows} rows")
+
+
+def wkv(planes: torch.Tensor, z: torch.Tensor, w0: torch.Tensor, u: torch.Tensor, state: torch.Tensor, rows: StepRows,
+        n_heads: int, dim: int) -> torch.Tensor:
+    """Time mixing over a step's rows: per head ``o = (S + diag(u) k v^T)^T r``, then
+    ``S <- diag(w) S + k v^T`` with ``w = exp(-exp(z + w0))`` per key channel, from the state the
+    sequences' earlier steps left.  ``planes`` [>= 3, rows, heads * dim] holds r, k and v; ``z`` float32
+    [rows, heads * dim]; ``state`` float32 [slots, heads, dim (value), dim (key)] is read and updated.
+    Returns the read-out, float32 [rows, heads, dim]."""
+    _wkv_check(planes, w0, u, state, rows, n_heads, dim, "wkv")
+    _need(z, "wkv z", torch.float32)
+    if tuple(z.shape) != (rows.n_rows, n_heads * dim):
+        raise KernelError(f"wkv: z {tuple(z.shape)}")
+    o = torch.empty((rows.n_rows, n_heads, dim), dtype=torch.float32, device=planes.device)
+    scratch = torch.empty(lib().thn_wkv_scratch_floats(rows.n_rows, n_heads, dim), dtype=torch.float32, device=planes.device)
+    _call("thn_wkv", _ptr(o), _ptr(state), _ptr(scratch), _ptr(planes[0]), _ptr(planes[1]), _ptr(planes[2]), _ptr(z), _ptr(w0),
+          _ptr(u), _ptr(rows.cu_seqlens), _ptr(rows.slots), rows.n_rows, rows.n_seqs, n_heads, dim, _code(planes, "wkv"), _stream())
+    return o
+
+
+def wkv_decode(planes: torch.Tensor, low: torch.Tensor, w2: torch.Tensor, w0: torch.Tensor, u: torch.Tensor, gain: torch.Tensor,
+               eps: float, state: torch.Tensor, rows: StepRows, n_heads: int, dim: int) -> torch.Tensor:
+    """One token per sequence, all of time mixing between the first products and the last: ``planes``
+    [4, rows, heads * dim] holds r, k, v and the gate's input; the decay's input is
+    ``w2 tanh(low) + w0`` with ``low`` float32 [rows, rank] and ``w2`` [heads * dim, rank]; the read-out
+    of a head is divided by its root mean square, times ``gain`` (float32 [heads * dim]), times silu of
+    the gate.  Returns [rows, heads * dim] of the activation type."""
+    _wkv_check(planes, w0, u, state, rows, n_heads, dim, "wkv_decode")
+    _need(low, "wkv_decode low", torch.float32)
+    _need(w2, "wkv_decode w2", planes.dtype)
+    _need(gain, "wkv_decode gain", torch.float32)
+    if planes.shape[0] < 4 or rows.max_q_len != 1 or low.shape[0] != rows.n_rows \
+            or tuple(w2.shape) != (n_heads * dim, low.shape[1]) or gain.shape[0] != n_heads * dim:
+        raise KernelError(f"wkv_decode: projections {tuple(planes.shape)}, low {tuple(low.shape)}, w2 {tuple(w2.shape)}")
+    out = torch.empty((rows.n_rows, n_heads * dim), dtype=planes.dtype, device=planes.device)
+    _call("thn_wkv_decode", _ptr(out), _ptr(state), _ptr(planes[0]), _ptr(planes[1]), _ptr(planes[2]), _ptr(planes[3]), _ptr(low),
+          low.shape[1], _ptr(w2), _ptr(w0), _ptr(u), _ptr(gain), float(eps), _ptr(rows.row_slot), rows.n_rows, n_heads, dim,
+          _code(planes, "wkv_decode"), _stream())
+    return out
+
+
+@dataclass
+class StateSpace:
+    """Sizes and float32 constants of a state-space-duality mixer.  The convolution's channels are
+    ``[x: heads * vdim | B: groups * state | C: groups * state]``."""
+
+    n_heads: int
+    vdim: int
+    n_state: int
+    n_groups: int
+    conv_w: torch.Tensor      # [channels, taps], the last tap the current token's
+    conv_b: torch.Tensor      # [channels]
+    dt_bias: torch.Tensor     # [heads]
+    rate: torch.Tensor        # [heads]: the decay is exp(-rate * step size)
+    skip: torch.Tensor        # [heads]
+
+    @property
+    def channels(self) -> int:
+        return self.n_heads * self.vdim + 2 * self.n_groups * self.n_state
+
+    @property
+    def taps(self) -> int:
+        return self.conv_w.shape[1]
+
+
+def state_space(proj: torch.Tensor, offset: int, dt_pre: torch.Tensor, shape: StateSpace, state: torch.Tensor,
+                ring: torch.Tensor, rows: StepRows, seq_lens: torch.Tensor) -> torch.Tensor:
+    """State-space duality over a step's rows: the short causal convolution (bias, silu) over the
+    columns ``[offset, offset + channels)`` of ``proj``, step sizes ``t = softplus(dt_pre + dt_bias)`` and
+    decays ``a = exp(-rate t)`` per head, then ``S <- a S + (t B) x^T``, ``y = S^T C + skip x`` per head (B
+    and C of the head's group).  ``state`` float32 [slots, heads, vdim, state] and ``ring``
+    [slots, taps, channels] (position p at ``p mod taps``) are read and updated; ``seq_lens`` holds the
+    tokens each slot held before the step.  Returns y float32 [rows, heads, vdim].  Steps of one token
+    per sequence run as one kernel, others as three (prepare, recurrence, ring update)."""
+    _need(proj, "state_space proj")
+    _need(dt_pre, "state_space dt", torch.float32)
+    _need(state, "state_space state", torch.float32)
+    _need(ring, "state_space ring", proj.dtype)
+    s, n = shape, rows.n_rows
+    for t, what, want in ((s.conv_w, "conv", (s.channels, s.taps)), (s.conv_b, "conv bias", (s.channels,)),
+                          (s.dt_bias, "dt bias", (s.n_heads,)), (s.rate, "rate", (s.n_heads,)), (s.skip, "skip", (s.n_heads,))):
+        _need(t, f"state_space {what}", torch.float32)
+        if tuple(t.shape) != want:
+            raise KernelError(f"state_space: {what} is {tuple(t.shape)}, expected {want}")
+    if proj.shape[0] != n or tuple(dt_pre.shape) != (n, s.n_heads) or tuple(state.shape[1:]) != (s.n_heads, s.vdim, s.n_state) \
+            or tuple(ring.shape[1:]) != (s.taps, s.channels) or ring.shape[0] != state.shape[0]:
+        raise KernelError(f"state_space: proj {tuple(proj.shape)}, dt {tuple(dt_pre.shape)}, state {tuple(state.shape)}, ring "
+                          f"{tuple(ring.shape)} do not fit {s.n_heads} heads of {s.n_state} x {s.vdim} over {n} rows")
+    y = torch.empty((n, s.n_heads, s.vdim), dtype=torch.float32, device=proj.device)
+    code = _code(proj, "state_space")
+    if rows.max_q_len == 1:
+        _call("thn_state_space_decode", _ptr(y), _ptr(state), _ptr(proj), proj.shape[1], int(offset), _ptr(s.conv_w),
+              _ptr(s.conv_b), _ptr(ring), _ptr(dt_pre), _ptr(s.dt_bias), _ptr(s.rate), _ptr(s.skip), _ptr(rows.row_slot),
+              _ptr(rows.row_pos), n, s.n_heads, s.vdim, s.n_state, s.n_groups, s.taps, code, _stream())
+        return y
+    scratch = torch.empty(lib().thn_state_space_scratch_floats(n, s.n_heads, s.vdim, s.n_state, s.n_groups), dtype=torch.float32,
+                          device=proj.device)
+    _call("thn_state_space", _ptr(y), _ptr(state), _ptr(scratch), _ptr(proj), proj.shape[1], int(offset), _ptr(s.conv_w),
+          _ptr(s.conv_b), _ptr(ring), _ptr(dt_pre), _ptr(s.dt_bias), _ptr(s.rate), _ptr(s.skip), _ptr(rows.row_slot),
+          _ptr(rows.row_pos), _ptr(seq_lens), _ptr(rows.cu_seqlens), _ptr(rows.slots), n, rows.n_seqs, s.n_heads, s.vdim,
+          s.n_state, s.n_groups, s.taps, code, _stream())
+    conv_ring_update(ring, proj, offset, rows, seq_lens)
+    return y
+
+
+def gated_group_norm(y: torch.Tensor, gate: torch.Tensor, gate_offset: int, gain: torch.Tensor, eps: float, parts: int,
+                     dtype: torch.dtype) -> torch.Tensor:
+    """y float32 [rows, ...] (``width`` entries a row) times silu of ``gate[:, gate_offset : gate_offset +
+    width]``, divided by its root mean square over each of ``parts`` equal consecutive parts, times ``gain``
+    (float32 [width]) -> [rows, width] of ``dtype``: a gate ahead of the norm."""
+    _need(y, "gated_group_norm y", torch.float32)
+    _need(gate, "gated_group_norm gate", dtype)
+    _need(gain, "gated_group_norm gain", torch.float32)
+    rows = y.shape[0]
+    width = gain.shape[0]
+    if y.numel() != rows * width or width % parts or gate.shape[0] != rows or gate_offset + width > gate.shape[1]:
+        raise KernelError(f"gated_group_norm: y {tuple(y.shape)}, gate {tuple(gate.shape)} from {gate_offset}, gain of {width}, "
+                          f"{parts} parts")
+    out = torch.empty((rows, width), dtype=dtype, device=y.device)
+    _call("thn_gated_group_norm", _ptr(out), _ptr(y), gate.data_ptr() + gate_offset * gate.element_size(), gate.shape[1],
+          _ptr(gain), float(eps), rows, width, int(parts), DTYPE_CODE[dtype], _stream())
+    return out
+
+
 def rotate_gate(a: torch.Tensor, gate: torch.Tensor, gate_offset: int, n_heads: int, size: int,
                 rotary: Optional[RotaryTables], rows: StepRows, err: Optional[torch.Tensor], scale: float = 1.0,
                 out: Optional[torch.Tensor] = None, out_offset: int = 0) -> torch.Tensor:
@@ -1583,5 +1839,5 @@ def gather_i32(src: torch.Tensor, index: torch.Tensor, out: Optional[torch.Tenso
 __all__ = [
     "KernelError", "KernelLibraryError", "KVView", "RotaryTables", "RowTiles", "StepRows", "row_tiles_of", "prompt_attention_tile", "linear_stream", "linear_swiglu", "linear_tcgen05", "add_rmsnorm", "advance",
     "ROW_TILE", "attention", "attention_decode_bf16", "attention_generic", "attention_prefill_bf16", "attention_prefill_tcgen05", "decode_splits", "choose_tokens", "gather_i32", "gather_rows", "lib", "linear", "new_error_word",
-    "qk_norm_rope_cache", "qk_prepare", "Gain", "STREAM_AS_IS", "residual_norm", "gather_rows_scaled", "logistic_gate", "latent_norm", "latent_assemble", "mlstm", "mlstm_column_blocks", "set_mlstm_kernel", "Routing", "moe_route", "routed_gelu", "gated_head_norm", "clamped_glu", "routed_clamped_glu", "polynorm", "scale_", "ScoreShape", "PLAIN_SCORES", "DeltaShape", "delta_rule", "qkv_attention", "raise_on_device_error", "rmsnorm", "StreamNumbers", "hyper_norm", "linear_attention", "causal_conv", "conv_ring_update", "selective_scan", "rotate_gate", "rope_table", "scatter_i32", "step_rows", "swiglu",
+    "qk_norm_rope_cache", "qk_prepare", "Gain", "STREAM_AS_IS", "residual_norm", "gather_rows_scaled", "logistic_gate", "latent_norm", "latent_assemble", "mlstm", "mlstm_column_blocks", "set_mlstm_kernel", "Routing", "moe_route", "routed_gelu", "gated_head_norm", "clamped_glu", "routed_clamped_glu", "polynorm", "scale_", "ScoreShape", "PLAIN_SCORES", "DeltaShape", "delta_rule", "qkv_attention", "raise_on_device_error", "rmsnorm", "StreamNumbers", "hyper_norm", "linear_attention", "causal_conv", "conv_ring_update", "selective_scan", "PairTable", "embed_rows", "squared_relu", "linear_batched", "token_shift", "tanh_rows", "wkv", "wkv_decode", "StateSpace", "state_space", "gated_group_norm", "rotate_gate", "rope_table", "scatter_i32", "step_rows", "swiglu",
 ]

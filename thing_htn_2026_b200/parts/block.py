@@ -1,7 +1,8 @@
 """Arrangement of a layer's parts.  ``pre_norm``: ``a = x + mixer(norm(x))``,
 ``y = a + ffn(norm(a))`` (OPTIMIZATION_GUIDE.md:57-70).  The add of a branch's output is
 deferred to the next norm, which fuses it (engine/engine.py:1104-1118): a block takes and
-returns the pair (residual stream ``h``, pending branch output ``d`` or None).
+returns the pair (residual stream ``h``, pending branch output ``d`` or None).  The feed-forward half
+may be absent; the stream is kept in whatever type the embedding starts it in.
 
 A block owns its sub-parts.  Their specs are parameters of the block's own spec, the block
 builds them, lists their tensors, answers for their cache need and passes on what they
@@ -97,6 +98,8 @@ class PreNormBlock(Block):
                 entry: ScheduleEntry) -> Tuple[torch.Tensor, torch.Tensor]:
         n = self.norm_mixer.forward(h) if d is None else self.norm_mixer.add_forward(h, d)
         a = self.mixer.forward(n, ctx, entry)
+        if self.ffn is None:
+            return h, a
         n = self.norm_ffn.add_forward(h, a)
         return h, self.ffn.forward(n, ctx)
 

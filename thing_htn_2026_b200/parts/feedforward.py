@@ -21,6 +21,8 @@ depend on the other rows of the step.  Kernels: csrc/moe.cu.
 taken entry by entry and ``N`` the division of a token's vector by its root mean square (``eps``
 inside the root); the four numbers are a tensor of the layer (``act``).
 
+``squared_relu``: ``down(max(up(x), 0)^2)``.
+
 ``routed_clamped_experts``: a mixture whose experts have the form of ``clamped_glu`` (``limit``,
 ``slope``).  Scores are ``logistic(router(x))``, each expert by itself, in float32; the ``top``
 largest are chosen and weighted by their scores as they are.  The weight multiplies the expert's
@@ -30,13 +32,19 @@ the projected values by ``w`` before the clamps; one down-projection over all ex
 sums the chosen ones.  With ``shared_ff`` a shared expert with a limit of its own
 (``shared_limit``) runs for every token on the token itself and is added times
 ``logistic(shared_gate(x))`` (``shared_gated`` False: added as it is).  ``scoring`` "softmax": the
-scores are a softmax over all experts instead; ``renormalise`` (a small number): the chosen
+scores are a softmax over all experts instead; "softmax_chosen": the largest logits are chosen and
+weighted by the softmax over the chosen logits alone; ``renormalise`` (a small number): the chosen
 experts' scores are divided by their sum plus that number; ``weight_at`` "output": an expert sees
 the token itself and its output is weighted (the weight then multiplies the activation, ahead of
-the one down-projection over all columns)."""
+the one down-projection over all columns).
+
+``routed_glu_experts``: the same with experts of the plain form ``down(silu(gate(x)) * up(x))``: the
+parameters default to no limit, slope 1, nothing added to the up branch (``up_shift`` 0 instead of 1),
+scores by a softmax over the chosen logits, the weight at the output and an ungated shared expert."""
 
 from __future__ import annotations
 
+import math
 from typing import List
 
 import torch
@@ -155,8 +163,27 @@ class PolyNormFFN:
         return ops.linear(ops.polynorm(ops.linear(x, self.w_up, err=err), self.coefficients, self.eps), self.w_down, err=err)
 
 
+@register_part("ffn", "squared_relu")
+class SquaredReluFFN:
+    @classmethod
+    def tensor_specs(cls, spec: PartSpec) -> List[TensorSpec]:
+        hidden, inter = int(spec.params["hidden_size"]), int(spec.params["intermediate_size"])
+        return [TensorSpec(spec.tensors["up_proj"], (inter, hidden), MATRIX),
+                TensorSpec(spec.tensors["down_proj"], (hidden, inter), MATRIX)]
+
+    def __init__(self, spec: PartSpec, runtime: Runtime):
+        self.w_up = runtime.tensor(spec, "up_proj")
+        self.w_down = runtime.tensor(spec, "down_proj")
+
+    def forward(self, x: torch.Tensor, ctx) -> torch.Tensor:
+        err = getattr(ctx, "err", None)
+        return ops.linear(ops.squared_relu(ops.linear(x, self.w_up, err=err)), self.w_down, err=err)
+
+
 @register_part("ffn", "routed_clamped_experts")
 class RoutedClampedExperts:
+    DEFAULTS = {}     # parameters that a form of expert fixes where the spec does not name them
+
     @staticmethod
     def _sizes(spec: PartSpec):
         p = spec.params
@@ -174,18 +201,19 @@ class RoutedClampedExperts:
             specs += [TensorSpec(spec.tensors["shared_gate_proj"], (shared, hidden), MATRIX),
                       TensorSpec(spec.tensors["shared_up"], (shared, hidden), MATRIX),
                       TensorSpec(spec.tensors["shared_down"], (hidden, shared), MATRIX)]
-            if spec.params.get("shared_gated", True):
+            if {**cls.DEFAULTS, **spec.params}.get("shared_gated", True):
                 specs.append(TensorSpec(spec.tensors["shared_gate"], (1, hidden), MATRIX))
         return specs
 
     def __init__(self, spec: PartSpec, runtime: Runtime):
-        p = spec.params
+        p = {**self.DEFAULTS, **spec.params}
         _, self.n_experts, self.ff, self.shared_ff = self._sizes(spec)
         self.top = int(p["top"])
         if not 0 < self.top <= self.n_experts:
             raise ValueError(f"routed_clamped_experts: top {self.top} of {self.n_experts} experts")
         self.limit, self.slope = float(p["limit"]), float(p["slope"])
         self.shared_limit = float(p.get("shared_limit") or self.limit)
+        self.up_shift = float(p.get("up_shift", 1.0))
         self.scoring = str(p.get("scoring", "logistic"))
         self.renormalise = None if p.get("renormalise") is None else float(p["renormalise"])
         self.weight_at = str(p.get("weight_at", "input"))
@@ -214,5 +242,11 @@ class RoutedClampedExperts:
         routing = ops.moe_route(z, self.n_experts, 1, 1, self.top, 1.0, scoring=self.scoring, renormalise=self.renormalise)
         gu = ops.linear(x, self.w_gate_up, err=err)
         y = ops.routed_clamped_glu(gu, routing, self.ff, self.shared_ff, self.limit, self.shared_limit, self.slope,
-                                   z if self.shared_gated else None, self.n_experts, weight_at=self.weight_at)
+                                   z if self.shared_gated else None, self.n_experts, weight_at=self.weight_at, up_shift=self.up_shift)
         return ops.linear(y, self.w_down, err=err)
+
+
+@register_part("ffn", "routed_glu_experts")
+class RoutedGLUExperts(RoutedClampedExperts):
+    DEFAULTS = {"limit": math.inf, "slope": 1.0, "up_shift": 0.0, "scoring": "softmax_chosen", "weight_at": "output",
+                "shared_gated": False}

@@ -11,9 +11,11 @@ entries per head, values of ``value_dim`` and a latent of ``latent_rank``:
     score        = (q_h . k_h) * scale        with the rot part of q_h rotated as well
     out          = W_o (concat_h softmax(score) v_h * logistic(W_g x))
 
-The rotation pairs entries 2i and 2i + 1 of the rot part (the position part's "interleaved"
-layout, with whatever frequency scaling its spec names).  ``window`` (None: all keys): position
-i sees j with 0 <= i - j < window.  ``gated`` False leaves the output gate (and ``g_proj``) out.
+The rotation pairs the entries of the rot part as the position part's layout says ("interleaved"
+or "half"), with whatever frequency scaling its spec names.  ``window`` (None: all keys): position
+i sees j with 0 <= i - j < window.  ``gated`` False leaves the output gate (and ``g_proj``) out;
+``gate_scope`` "value" (the default): a gate per entry, as above; "head": one number per head,
+``W_g`` has ``n_heads`` rows and a head's output is multiplied by its gate.
 
 One product gives q, the latent row and the gate (weights concatenated ``[q; dkv; g]``); a
 second one, on the normalised latent, gives every head's unrotated key and value (``[uk; uv]``).
@@ -56,7 +58,8 @@ class LatentAttention:
                  TensorSpec(spec.tensors["up_k"], (h * d, c), MATRIX),
                  TensorSpec(spec.tensors["up_v"], (h * e, c), MATRIX)]
         if spec.params.get("gated", True):
-            specs.append(TensorSpec(spec.tensors["g_proj"], (h * e, hidden), MATRIX))
+            per_head = spec.params.get("gate_scope", "value") == "head"
+            specs.append(TensorSpec(spec.tensors["g_proj"], (h if per_head else h * e, hidden), MATRIX))
         specs.append(TensorSpec(spec.tensors["o_proj"], (hidden, h * e), MATRIX))
         return specs
 
@@ -69,6 +72,9 @@ class LatentAttention:
         self.window: Optional[int] = None if p.get("window") is None else int(p["window"])
         self.eps = float(p["norm_eps"])
         self.gated = bool(p.get("gated", True))
+        if p.get("gate_scope", "value") not in ("value", "head"):
+            raise ValueError(f"latent_attention: gate_scope {p.get('gate_scope')!r} is neither 'value' nor 'head'")
+        self.head_gate = p.get("gate_scope", "value") == "head"
         self.exact_weights = p.get("softmax_weights") == "float32"
         self.dtype = runtime.dtype
         # the size of a value in the cache and in the attention's output: its own, or the keys'
@@ -81,7 +87,7 @@ class LatentAttention:
         parts = [runtime.tensor(spec, "q_proj"), runtime.tensor(spec, "down_proj")]
         if self.gated:
             gate = runtime.tensor(spec, "g_proj")
-            if pad:
+            if pad and not self.head_gate:
                 gate = torch.nn.functional.pad(gate.view(self.n_heads, self.value_dim, hidden), (0, 0, 0, pad))
                 gate = gate.reshape(self.n_heads * self.out_dim, hidden)
             parts.append(gate)
@@ -136,5 +142,5 @@ class LatentAttention:
         a = ops.attention(q, ctx.rows, kv, self.n_heads, self.scale, self.window, ctx.err, tiles,
                           exact_weights=self.exact_weights)
         if self.gated:
-            a = ops.logistic_gate(a, proj, self.gate_offset)
+            a = ops.logistic_gate(a, proj, self.gate_offset, self.out_dim if self.head_gate else 1)
         return ops.linear(a, self.w_o, err=ctx.err)

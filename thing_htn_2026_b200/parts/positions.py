@@ -59,8 +59,6 @@ class Rope:
             exponent = torch.arange(0, self.rotary_dim, 2, dtype=torch.int64).to(torch.float32) / self.rotary_dim
             self.inv_freq = (1.0 / (self.theta ** exponent)).to(runtime.device)
         self.exact_angles = spec.params.get("angle_precision") == "float64"
-        if self.exact_angles and spec.params.get("scaling"):
-            raise ValueError("rope: angles in double are built without frequency scaling")
         self.inv_freq64 = (self.theta ** -(torch.arange(0, self.rotary_dim, 2, dtype=torch.int64).to(torch.float64)
                                            / self.rotary_dim)).to(runtime.device)
         self.magnitude = 1.0
@@ -77,7 +75,9 @@ class Rope:
             hi = min(math.ceil(turn(float(scaling["slow"]))), self.rotary_dim - 1)
             index = torch.arange(self.rotary_dim // 2, dtype=torch.float64)
             ramp = ((index - lo) / max(hi - lo, 0.001)).clamp(0.0, 1.0)
-            self.inv_freq = (plain / factor * ramp + plain * (1.0 - ramp)).to(torch.float32).to(runtime.device)
+            stretched = plain / factor * ramp + plain * (1.0 - ramp)
+            self.inv_freq = stretched.to(torch.float32).to(runtime.device)
+            self.inv_freq64 = stretched.to(runtime.device)
             self.magnitude = 0.1 * math.log(factor) + 1.0
         self.device = runtime.device
         self._tables = None
@@ -93,10 +93,11 @@ class Rope:
         sin = torch.empty((size, half), dtype=torch.float32, device=self.device)
         if self.exact_angles:
             angle = torch.arange(size, dtype=torch.float64, device=self.device)[:, None] * self.inv_freq64[None, :]
-            cos, sin = torch.cos(angle).to(torch.float32).contiguous(), torch.sin(angle).to(torch.float32).contiguous()
+            cos = (torch.cos(angle) * self.magnitude).to(torch.float32).contiguous()
+            sin = (torch.sin(angle) * self.magnitude).to(torch.float32).contiguous()
         else:
             ops.rope_table(cos, sin, self.inv_freq, 0, size)
-        if self.magnitude != 1.0:
+        if self.magnitude != 1.0 and not self.exact_angles:
             cos.mul_(self.magnitude)
             sin.mul_(self.magnitude)
         self._tables = ops.RotaryTables(cos, sin, self.rotary_dim, self.layout)

@@ -96,13 +96,29 @@ def _log_spread(t, generator, matrix_std, gain_std):
     return t.normal_(0.0, gain_std, generator=generator).add_(base)
 
 
+def _unit_interval(t, generator, matrix_std, gain_std):
+    """A blend of two rows: between the one and the other."""
+    return t.uniform_(0.0, 1.0, generator=generator)
+
+
+def _log_decay(t, generator, matrix_std, gain_std):
+    """Input of a decay exp(-exp(w)): from a memory of hundreds of tokens down to less than one."""
+    return t.uniform_(0.0, 1.0, generator=generator).mul_(6.5).sub_(6.0)
+
+
+def _step_bias(t, generator, matrix_std, gain_std):
+    """Bias of a step size ahead of its softplus: steps between 0.01 and 0.7."""
+    return t.uniform_(0.0, 1.0, generator=generator).mul_(4.6).sub_(4.6)
+
+
 # How a tensor is drawn, by the name in ``TensorSpec.init``.  ``fill(t, generator, matrix_std,
 # gain_std)`` fills ``t`` (float32 on the CPU, the held dtype on a device) in place.
 INITIALIZERS: Dict[str, Callable] = {"normal": _normal, "one_plus_normal": _one_plus_normal, "zeros": _zeros,
                                      "zero_centered": _zero_centered, "conv_taps": _conv_taps, "log_rate": _log_rate,
                                      "unit_normal": _unit_normal, "small_normal": _small_normal, "gate_bias": _gate_bias, "polynomial": _polynomial,
                                      "stream_read": _stream_read, "stream_mix": _stream_mix, "sink": _sink,
-                                     "log_spread": _log_spread}
+                                     "log_spread": _log_spread, "unit_interval": _unit_interval,
+                                     "log_decay": _log_decay, "step_bias": _step_bias}
 # The rule of a spec that names none, by its role.
 ROLE_INIT = {MATRIX: "normal", GAIN: "one_plus_normal", TABLE: "zeros"}
 
