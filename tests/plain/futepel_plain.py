@@ -173,8 +173,9 @@ def latent_attention(ar, h, w, prefix, m, eps, positions):
     latent = ar.rb(rms_divide(down[:, :c], eps) * w[prefix + "dkv.norm"].to(ar.work))
     k_plain = ar.linear(latent, w[prefix + "uk"]).reshape(T, H, d)
     v = ar.linear(latent, w[prefix + "uv"]).reshape(T, H, e)
-    q_rot = ar.rb(rotate(q[:, :, d:], positions, m["rot"]))
-    k_rot = ar.rb(rotate(down[:, c:], positions, m["rot"]))
+    rot = m["rot"] if r else {"dims": 0}
+    q_rot = ar.rb(rotate(q[:, :, d:], positions, rot))
+    k_rot = ar.rb(rotate(down[:, c:], positions, rot))
     visible = positions[:, None] >= positions[None, :]
     out = torch.zeros(T, H, e, dtype=ar.work)
     for head in range(H):
