@@ -36,7 +36,10 @@ width, depth, heads and feed-forward products.  ``--design dubazen`` measures th
 (``dubazen-w2048``, ``dubazen-w4096``: four copies of the stream joined by hyper-connections, selective
 scans, pairs of softmax attention with sinks and linear attention, gated linear attention, routed
 experts weighted at their output) beside a Bunudra decoder of the same width, depth, heads and
-experts, its closest relative here.  The default run is untouched by all four.
+experts, its closest relative here.  ``--design futepel`` measures the Futepel decoder
+(``futepel-w2048``, ``futepel-w4096``: state-space duality, time mixing and latent attention over a plain
+float32 stream, dense squared-relu and routed feed-forwards) beside a Bunudra decoder of the same
+width, depth, latent attention and feed-forward weights.  The default run is untouched by all five.
 """
 
 from __future__ import annotations
@@ -1282,6 +1285,257 @@ def dubazen_kernel_table(torch, dub, peak, batch, context):
     return rows
 
 
+FUTEPEL_SIZES = ("futepel-w2048", "futepel-w4096")
+
+
+def bunudra_like_futepel(fut):
+    """A Bunudra config.json of the same width, depth and vocabulary as a Futepel configuration: a
+    matrix-memory layer (width / 128 heads of 128 x 128) for every time-mixing or state-space layer, the
+    same latent attention, and experts with the same number of weights as each layer's feed-forward."""
+    W = fut["width"]
+    layers = []
+    for layer in fut["layers"]:
+        mlp, m = layer["mlp"], layer["mixer"]
+        if mlp["kind"] == "dense":           # up and down; here eight experts of up and down, one of them shared
+            experts, ff, top = 7, mlp["ff"] // 8, 2
+        else:                                # gate, up and down; here up and down, half again as wide
+            experts, ff, top = mlp["router"]["experts"], mlp["expert"]["ff"] * 3 // 2, mlp["router"]["top"]
+        moe = {"kind": "moe", "expert": {"ff": ff}, "router": {"experts": experts, "top": top, "scale": 1.0}, "shared": {"ff": ff}}
+        if layer["type"] == "latent_attention":
+            kind, mixer = "latent_attention", {k: m[k] for k in ("heads", "dim", "rot_dim", "vdim", "kv_rank", "scale", "rot")}
+        else:
+            kind, mixer = "mlstm", {"heads": W // 128, "dim": 128, "vdim": 128, "gate_cap": 15.0}
+        layers.append({"type": kind, "mixer": mixer, "mlp": moe})
+    return {"architecture": "Bunudra", "vocab": fut["vocab"], "width": W, "embedding": {"scale": fut["embedding"]["scale"]},
+            "norm": fut["norm"], "layers": layers}
+
+
+class KernelTable:
+    """Kernels timed alone with cold caches (a buffer larger than L2 is written between timed launches):
+    microseconds, and the fraction of the roofline that a kernel's algorithmic bytes or flops amount to."""
+
+    def __init__(self, torch, peak):
+        self.torch, self.rows = torch, {}
+        self.flush = torch.empty(256 << 20, dtype=torch.uint8, device="cuda:0")
+        self.hbm, self.tensor = peak["hbm_gbs"] * 1e9, peak["bf16_tflops"] * 1e12
+        self.cores = FP32_CORE_TFLOPS * 1e12
+
+    def timed(self, fn, reps=9):
+        torch, out = self.torch, []
+        for _ in range(reps):
+            self.flush.zero_()
+            start, end = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+            start.record()
+            fn()
+            end.record()
+            torch.cuda.synchronize()
+            out.append(start.elapsed_time(end) * 1e3)
+        return statistics.median(out[2:])
+
+    def row(self, name, fn, nbytes=0, flops=0, flop_peak=None, like=None):
+        us = self.timed(fn)
+        by_bytes, by_flops = nbytes / self.hbm, flops / (flop_peak or self.tensor)
+        t_roof = max(by_bytes, by_flops) * 1e6
+        self.rows[name] = {"us": round(us, 2), "roofline_us": round(t_roof, 3), "frac": round(t_roof / us, 5), "like": like,
+                           "bound": "hbm" if by_bytes >= by_flops else "flops", "exact_frac": t_roof / us}
+
+    def finished(self):
+        for r in self.rows.values():
+            if r["like"] in self.rows:
+                r["times_farther_than_like"] = round(self.rows[r["like"]]["exact_frac"] / r["exact_frac"], 2)
+        for r in self.rows.values():
+            del r["exact_frac"]
+        return self.rows
+
+
+def futepel_kernel_table(torch, fut, peak, batch, context):
+    """Every kernel of the Futepel design alone, beside the like kernel of the designs that have one: the
+    matrix memory, latent attention and experts of Bunudra, and the linear attention, scan and read-out
+    norms of Dubazen, at the heads that those designs have at this width."""
+    from thing_htn_2026_b200 import ops
+    from thing_htn_2026_b200.cache import KVSpec, SequenceCache, StateSpec
+    dev, bf = "cuda:0", torch.bfloat16
+    pick = lambda kind: next(l for l in fut["layers"] if l["type"] == kind)["mixer"]
+    wk, lat, ssm = pick("wkv"), pick("latent_attention"), pick("mamba2")
+    mlp = next(l["mlp"] for l in fut["layers"] if l["mlp"]["kind"] == "moe")
+    dense = next(l["mlp"] for l in fut["layers"] if l["mlp"]["kind"] == "dense")
+    W, T, V = fut["width"], PREFILL_TOKENS, fut["vocab"]
+    E, ff, sff, top = mlp["router"]["experts"], mlp["expert"]["ff"], mlp["shared"]["ff"], mlp["router"]["top"]
+    table = KernelTable(torch, peak)
+    row, cores = table.row, table.cores
+    g = torch.Generator(device=dev).manual_seed(0)
+    rnd = lambda *shape: torch.randn(shape, generator=g, device=dev)
+    err = ops.new_error_word(dev)
+    n_slots = batch + 1
+    h, d, rank = wk["heads"], wk["dim"], wk["rank"]
+    H2, e2, N, G2, taps, parts = ssm["heads"], ssm["vdim"], ssm["state"], ssm["groups"], ssm["conv"], ssm["norm_groups"]
+    Hg, dg = W // 128, 128                      # heads of the like recurrences at this width
+    inner, scan_state = 2 * W, 16
+    channels = H2 * e2 + 2 * G2 * N
+    cache = SequenceCache([(StateSpec((h, d, d)), StateSpec((W,), bf)), (StateSpec((H2, e2, N)), StateSpec((taps, channels), bf)),
+                           StateSpec((Hg, dg, dg)), (StateSpec((inner, scan_state)), StateSpec((taps, inner), bf))],
+                          max_tokens=n_slots * 64, dtype=bf, device=dev, max_slots=n_slots + 1)
+    slots = cache.open(n_slots)
+    previous = cache.sequence_state("previous_token")
+    emb, buckets = rnd(V, W).to(bf), fut["embedding"]["bigram"]["buckets"]
+    pairs = ops.PairTable(rnd(buckets + 1, W).to(bf), fut["embedding"]["bigram"]["mul_prev"], fut["embedding"]["bigram"]["mul_cur"])
+    places = rnd(8192, W).to(bf)
+    mu, w_wide = torch.rand(5, W, device=dev), rnd(4, h * d, W).to(bf) * 0.02
+    w_one = rnd(4 * h * d, W).to(bf) * 0.02
+    w1, w2 = rnd(rank, W).to(bf) * 0.02, rnd(h * d, rank).to(bf) * 0.1
+    w0, u, gain_w = torch.rand(h * d, device=dev) * 4 - 5, rnd(h, d), 1 + rnd(h * d) * 0.1
+    shape = ops.StateSpace(H2, e2, N, G2, rnd(channels, taps) * 0.5, rnd(channels) * 0.1, rnd(H2) - 3.0,
+                           torch.rand(H2, device=dev) * 8 + 0.5, 1 + rnd(H2) * 0.1)
+    gain_s, gain_g = 1 + rnd(H2 * e2) * 0.1, 1 + rnd(dg) * 0.1
+    gate_bias = rnd(Hg * dg) + 3.0
+    conv_w, conv_b = rnd(inner, taps) * 0.5, rnd(inner) * 0.1
+    a_neg, d_skip, dt_bias = -torch.exp(rnd(inner, scan_state) * 0.5), 1 + rnd(inner) * 0.1, rnd(inner) * 0.1
+    for n, who, tag in ((T, slots[:1], "prefill"), (1, slots[1:], "decode")):
+        cu = torch.arange(len(who) + 1, dtype=torch.int32, device=dev) * n
+        m = n * len(who)
+        rows_ = ops.step_rows(cu, torch.tensor(who, dtype=torch.int32, device=dev), cache.seq_lens, m, n)
+        # ---- embedding, residual and norm, routing, activations, gates
+        tokens = torch.randint(0, V, (m,), generator=g, device=dev, dtype=torch.int32)
+        row(f"{tag}: embed_rows (pairs, positions)",
+            lambda: ops.embed_rows(emb, tokens, 8.0, rows_, cache.seq_lens, pairs, previous, places, err), nbytes=m * W * 10,
+            like=f"{tag}: gather_rows_scaled")
+        row(f"{tag}: gather_rows_scaled", lambda: ops.gather_rows_scaled(emb, tokens, 8.0, err), nbytes=m * W * 6)
+        h32, d16 = rnd(m, W), rnd(m, W).to(bf)
+        rms = ops.Gain(1 + rnd(W) * 0.1, 0.0, 1e-6)
+        layer = ops.Gain(1 + rnd(W) * 0.1, 0.0, 1e-6, rnd(W) * 0.1, "layer")
+        row(f"{tag}: residual_norm (add, RMS norm)", lambda: ops.residual_norm(h32, d16, None, rms, bf), nbytes=m * W * 12,
+            like=f"{tag}: residual_norm (layer norm of the branch, add)")
+        row(f"{tag}: residual_norm (layer norm of the branch, add)",
+            lambda: ops.residual_norm(h32, d16, layer, ops.STREAM_AS_IS, bf), nbytes=m * W * 12)
+        z = rnd(m, E + 1)
+        routing = ops.moe_route(z, E, 1, 1, top, 1.0, scoring="softmax_chosen")
+        row(f"{tag}: moe_route (softmax over the chosen)", lambda: ops.moe_route(z, E, 1, 1, top, 1.0, scoring="softmax_chosen"),
+            nbytes=m * ((E + 1) * 4 + E * 4 + top * 8), like=f"{tag}: moe_route (softmax, groups)")
+        row(f"{tag}: moe_route (softmax, groups)", lambda: ops.moe_route(z, E, 4, 2, top, 2.0),
+            nbytes=m * ((E + 1) * 4 + E * 4 + top * 8))
+        gu, up = rnd(m, 2 * (E * ff + sff)).to(bf), rnd(m, E * ff + sff).to(bf)
+        row(f"{tag}: routed_clamped_glu (silu, no limit)",
+            lambda: ops.routed_clamped_glu(gu, routing, ff, sff, float("inf"), float("inf"), 1.0, weight_at="output", up_shift=0.0),
+            nbytes=m * (2 * (top * ff + sff) * 2 + (E * ff + sff) * 2), like=f"{tag}: routed_gelu")
+        row(f"{tag}: routed_gelu", lambda: ops.routed_gelu(up, routing, ff, sff, z, E),
+            nbytes=m * ((top * ff + sff) * 2 + (E * ff + sff) * 2))
+        wide = rnd(m, dense["ff"]).to(bf)
+        row(f"{tag}: squared_relu", lambda: ops.squared_relu(wide), nbytes=m * dense["ff"] * 4, like=f"{tag}: clamped_glu")
+        row(f"{tag}: clamped_glu", lambda: ops.clamped_glu(wide, 7.0, 1.702), nbytes=m * dense["ff"] * 3)
+        Hl, El = lat["heads"], lat["vdim"]
+        a16, g16 = rnd(m, Hl * El).to(bf), rnd(m, Hl * El + 64).to(bf)
+        row(f"{tag}: logistic_gate (per head)", lambda: ops.logistic_gate(a16, g16, 64, El), nbytes=m * Hl * (El * 4 + 2),
+            like=f"{tag}: logistic_gate")
+        row(f"{tag}: logistic_gate", lambda: ops.logistic_gate(a16, g16, 64), nbytes=m * Hl * El * 6)
+        # ---- time mixing
+        shift, state = cache.state_view(0, 1), cache.state_view(0, 0)
+        row(f"{tag}: token_shift (five blends)", lambda: ops.token_shift(d16, mu, shift, rows_, cache.seq_lens),
+            nbytes=m * W * 12, like=f"{tag}: logistic_gate")
+        blends = ops.token_shift(d16, mu, shift, rows_, cache.seq_lens)
+        prod = dict(flops=8.0 * m * W * h * d, nbytes=4 * W * h * d * 2)
+        row(f"{tag}: linear_batched (r, k, v, gate)", lambda: ops.linear_batched(blends[:4], w_wide),
+            like=f"{tag}: linear (one product of the same size)", **prod)
+        row(f"{tag}: linear (one product of the same size)", lambda: ops.linear(d16, w_one, err=err), **prod)
+        row(f"{tag}: linear (decay, first)", lambda: ops.linear(blends[4], w1, out_dtype=torch.float32, err=err),
+            flops=2.0 * m * W * rank, nbytes=W * rank * 2 + m * (W * 2 + rank * 4))
+        planes, low = (rnd(4, m, h * d) * 0.5).to(bf), rnd(m, rank)
+        lin = rnd(m, Hg * 4 * dg).to(bf) * 0.5
+        zg = rnd(m, Hg * dg)
+        state_bytes, like_state = len(who) * h * d * d * 8, len(who) * Hg * dg * dg * 8
+        like_la = f"{tag}: linear_attention (gated decays)"
+        la = lambda: ops.linear_attention(lin, (0, Hg * dg, 2 * Hg * dg), cache.state_view(2), rows_, Hg, dg, dg, gate=zg,
+                                          gate_bias=gate_bias, tau=16.0, q_scale=dg ** -0.5)
+        row(like_la, la, nbytes=like_state + m * Hg * dg * (3 * 2 + 4 + 4), flops=6.0 * m * Hg * dg * dg, flop_peak=cores)
+        o_like = rnd(m, Hg, dg)
+        row(f"{tag}: gated_head_norm (one gain)", lambda: ops.gated_head_norm(o_like, lin, 3 * Hg * dg, gain_g, 1e-6, Hg, dg, bf),
+            nbytes=m * Hg * dg * 8)
+        if tag == "prefill":
+            zt = ops.linear(ops.tanh_rows(low, bf), w2, out_dtype=torch.float32, err=err)
+            row("prefill: tanh_rows", lambda: ops.tanh_rows(low, bf), nbytes=m * rank * 6, like="prefill: moe_route (softmax, groups)")
+            row("prefill: linear (decay, second)", lambda: ops.linear(ops.tanh_rows(low, bf), w2, out_dtype=torch.float32, err=err),
+                flops=2.0 * m * rank * h * d, nbytes=m * h * d * 4)
+            row("prefill: wkv (decays, recurrence)", lambda: ops.wkv(planes, zt, w0, u, state, rows_, h, d),
+                nbytes=state_bytes + m * h * d * (3 * 2 + 4 + 4), flops=6.0 * m * h * d * d, flop_peak=cores, like=like_la)
+            o32 = rnd(m, h, d)
+            row("prefill: gated_head_norm (a gain per head)",
+                lambda: ops.gated_head_norm(o32, planes[3], 0, gain_w, 1e-6, h, d, bf), nbytes=m * h * d * 8,
+                like="prefill: gated_head_norm (one gain)")
+        else:
+            row("decode: linear_attention (gated decays) + gated_head_norm",
+                lambda: (la(), ops.gated_head_norm(o_like, lin, 3 * Hg * dg, gain_g, 1e-6, Hg, dg, bf)),
+                nbytes=like_state + m * Hg * dg * (3 * 2 + 4 + 4 + 8), flops=6.0 * m * Hg * dg * dg, flop_peak=cores)
+            row("decode: wkv_decode (decay's second product, recurrence, norm, gate)",
+                lambda: ops.wkv_decode(planes, low, w2, w0, u, gain_w, 1e-6, state, rows_, h, d),
+                nbytes=state_bytes + m * h * d * 5 * 2 + h * d * rank * 2, flops=6.0 * m * h * d * d, flop_peak=cores,
+                like="decode: linear_attention (gated decays) + gated_head_norm")
+        # ---- state-space duality
+        proj, dt = rnd(m, H2 * e2 + channels).to(bf), rnd(m, H2)
+        row(f"{tag}: state_space (convolution, decays, recurrence, ring)",
+            lambda: ops.state_space(proj, H2 * e2, dt, shape, cache.state_view(1, 0), cache.state_view(1, 1), rows_, cache.seq_lens),
+            nbytes=len(who) * H2 * e2 * N * 8 + m * (channels * 2 + H2 * e2 * 4), flops=6.0 * m * H2 * e2 * N, flop_peak=cores,
+            like=like_la)
+        y32 = rnd(m, H2, e2)
+        row(f"{tag}: gated_group_norm", lambda: ops.gated_group_norm(y32, proj, 0, gain_s, 1e-6, parts, bf), nbytes=m * H2 * e2 * 8,
+            like=f"{tag}: gated_head_norm (one gain)")
+        xz, xc, dt_pre, bc = rnd(m, 2 * inner).to(bf), rnd(m, inner).to(bf), rnd(m, inner), rnd(m, 2 * scan_state).to(bf)
+        row(f"{tag}: causal_conv, its ring and selective_scan",
+            lambda: (ops.causal_conv(xz, 0, inner, conv_w, conv_b, cache.state_view(3, 1), rows_, cache.seq_lens),
+                     ops.conv_ring_update(cache.state_view(3, 1), xz, 0, rows_, cache.seq_lens),
+                     ops.selective_scan(xc, dt_pre, dt_bias, bc, a_neg, d_skip, xz, inner, cache.state_view(3, 0), rows_)),
+            nbytes=len(who) * inner * scan_state * 8 + m * inner * (2 + 2 + 4 + 2 + 2), flops=6.0 * m * inner * scan_state, flop_peak=cores)
+
+    # ---- latent attention over a paged cache: half pairs beside interleaved ones
+    Hl, P, R, El, C = lat["heads"], lat["dim"], lat["rot_dim"], lat["vdim"], lat["kv_rank"]
+    D = P + R
+    for layout, like in (("interleaved", False), ("half", True)):
+        tables = ops.RotaryTables(torch.ones(8192, R // 2, device=dev), torch.zeros(8192, R // 2, device=dev), R, layout)
+        kv = SequenceCache([KVSpec(Hl, D, None, 0, None, El)], max_tokens=(batch * (context + 64) + T + 64), dtype=bf, device=dev,
+                           max_slots=batch + 2)
+        own = kv.open(batch + 1)
+
+        def step_of(slot_list, counts):
+            kv.prepare(slot_list, counts)
+            cu = [0]
+            for c in counts:
+                cu.append(cu[-1] + c)
+            cu_dev, slots_dev = torch.tensor(cu, dtype=torch.int32, device=dev), torch.tensor(slot_list, dtype=torch.int32, device=dev)
+            return ops.step_rows(cu_dev, slots_dev, kv.seq_lens, cu[-1], max(counts),
+                                 max_context=max(kv.length(s) + c for s, c in zip(slot_list, counts)), lengths_differ=False), cu_dev, slots_dev
+
+        def prepare(proj, up, rows_):
+            ops.latent_norm(proj, Hl * D, C, gain_c, 1e-6)
+            return ops.latent_assemble(proj, 0, Hl * D + C, up, tables, rows_, kv.kv_view(0), Hl, P, R, err)
+
+        gain_c = 1 + rnd(C) * 0.1
+        width, up_width = Hl * D + C + R + Hl, Hl * (P + El)
+        per_row = (Hl * D + 2 * C + R + up_width) * 2 + (Hl * D + Hl * (D + El)) * 2
+        for n, who, tag in ((T, own[:1], "prefill"), (1, own[1:], "decode")):
+            if tag == "decode":
+                rows_, cu_dev, slots_dev = step_of(who, [context] * batch)
+                prepare(rnd(batch * context, width).to(bf), rnd(batch * context, up_width).to(bf), rows_)
+                ops.advance(kv.seq_lens, slots_dev, cu_dev)
+                kv.commit(who, [context] * batch)
+            rows_, cu_dev, slots_dev = step_of(who, [n] * len(who))
+            m = n * len(who)
+            proj, up = rnd(m, width).to(bf), rnd(m, up_width).to(bf)
+            row(f"{tag}: latent_norm + latent_assemble ({layout} pairs)", lambda: prepare(proj, up, rows_), nbytes=m * per_row,
+                like=f"{tag}: latent_norm + latent_assemble (interleaved pairs)" if like else None)
+            if not like:
+                continue
+            q = prepare(proj, up, rows_)
+            tiles, size = None, ops.prompt_attention_tile(bf, D, 64, Hl, Hl, El) if n > 1 else 0
+            if size:
+                r0, rn = ops.row_tiles_of([n], [0], size)
+                tiles = ops.RowTiles(torch.tensor(r0, dtype=torch.int32, device=dev), torch.tensor(rn, dtype=torch.int32, device=dev),
+                                     len(r0), size)
+            cost = dict(flops=2.0 * Hl * (D + El) * T * (T + 1) / 2, nbytes=T * Hl * (D + El) * 2) if n > 1 else \
+                dict(nbytes=batch * Hl * (context + 1) * (D + El) * 2)
+            row(f"{tag}: attention (latent heads, all keys; the kernel Bunudra's run)",
+                lambda: ops.attention(q, rows_, kv.kv_view(0), Hl, lat["scale"], None, err, tiles, exact_weights=True), **cost)
+    ops.raise_on_device_error(err, "kernel table")
+    return table.finished()
+
+
 def run_design(args):
     import torch
     from thing_htn_2026_b200 import Engine, ops
@@ -1294,7 +1548,8 @@ def run_design(args):
     sampler.start()
     ops.launch_count = 0
     design = args.design
-    design_sizes = {"lanilix": DESIGN_SIZES, "bunudra": BUNUDRA_SIZES, "ditilix": DITILIX_SIZES, "dubazen": DUBAZEN_SIZES}[design]
+    design_sizes = {"lanilix": DESIGN_SIZES, "bunudra": BUNUDRA_SIZES, "ditilix": DITILIX_SIZES, "dubazen": DUBAZEN_SIZES,
+                    "futepel": FUTEPEL_SIZES}[design]
     for name in design_sizes:
         lan = named_config_json(name)
         if args.layers:
@@ -1305,7 +1560,8 @@ def run_design(args):
         beside = {"lanilix": lambda: ("qwen3_same_size", qwen3_like(lan)),
                   "bunudra": lambda: ("lanilix_same_size", lanilix_like(lan)),
                   "ditilix": lambda: ("qwen3_same_size", qwen3_like_ditilix(lan)),
-                  "dubazen": lambda: ("bunudra_same_size", bunudra_like(lan))}[design]()
+                  "dubazen": lambda: ("bunudra_same_size", bunudra_like(lan)),
+                  "futepel": lambda: ("bunudra_same_size", bunudra_like_futepel(lan))}[design]()
         for label, data in ((design, lan), beside):
             engine = Engine.from_config(config_from_dict(data), seed=0, dtype="bfloat16", max_tokens=max_tokens,
                                         max_batch=args.batch)
@@ -1314,7 +1570,7 @@ def run_design(args):
             del engine
             torch.cuda.empty_cache()
         table = {"lanilix": kernel_table, "bunudra": bunudra_kernel_table, "ditilix": ditilix_kernel_table,
-                 "dubazen": dubazen_kernel_table}[design]
+                 "dubazen": dubazen_kernel_table, "futepel": futepel_kernel_table}[design]
         entry["kernels"] = table(torch, lan, peak, args.batch, args.prompt_len)
         sizes[name] = entry
     clocks = sampler.stop()
@@ -1529,9 +1785,9 @@ def main():
                              "(for ncu --profile-from-start off)")
     parser.add_argument("--workload", choices=sorted(LARGE_WORKLOADS), default=None,
                         help="one of the two larger workloads instead of the default run")
-    parser.add_argument("--design", choices=["lanilix", "bunudra", "ditilix", "dubazen"], default=None,
+    parser.add_argument("--design", choices=["lanilix", "bunudra", "ditilix", "dubazen", "futepel"], default=None,
                         help="another design beside its closest relative at the same sizes (Lanilix beside Qwen3, "
-                             "Bunudra beside Lanilix, Ditilix beside Qwen3), model by model and kernel by kernel, "
+                             "Bunudra beside Lanilix, Ditilix beside Qwen3, Dubazen and Futepel beside Bunudra), model by model and kernel by kernel, "
                              "instead of the default run")
     args = parser.parse_args()
     args.steps_given = args.steps is not None
