@@ -117,12 +117,21 @@ THN_API int thn_gather_rows_scaled(float* out, const void* table, const int* ind
 // sequence's first token takes row `buckets`, the table's last.  The token before the first row that a
 // sequence brings is what its last step left in `previous`; the block of that row leaves the step's last
 // token there, after it has read (no other block touches the slot).  pairs and positions may be null.
+template <typename T> __device__ __forceinline__ float4 four_of(const T* p);
+template <> __device__ __forceinline__ float4 four_of<float>(const float* p) { return *reinterpret_cast<const float4*>(p); }
+template <> __device__ __forceinline__ float4 four_of<__nv_bfloat16>(const __nv_bfloat16* p) {
+    const uint2 raw = *reinterpret_cast<const uint2*>(p);
+    const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.x));
+    const float2 b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.y));
+    return make_float4(a.x, a.y, b.x, b.y);
+}
+
 template <typename T>
 __global__ void embed_rows_kernel(float* __restrict__ out, const T* __restrict__ table, const int* __restrict__ tokens, int width,
                                   int n_table_rows, float scale, const T* __restrict__ pairs, int buckets, long long mul_before,
                                   long long mul_token, int* __restrict__ previous, const T* __restrict__ positions,
                                   int n_positions, const int* __restrict__ row_slot, const int* __restrict__ row_pos,
-                                  const int* __restrict__ cu_seqlens, const int* __restrict__ seq_lens, int n_seqs,
+                                  const int* __restrict__ cu_seqlens, const int* __restrict__ seq_lens, int n_seqs, int vec,
                                   int* __restrict__ err) {
     pdl_launch_dependents();
     pdl_wait();
@@ -161,6 +170,19 @@ __global__ void embed_rows_kernel(float* __restrict__ out, const T* __restrict__
     const T* pair = pairs != nullptr ? pairs + (size_t)pair_row * width : nullptr;
     const T* place = positions != nullptr ? positions + (size_t)pos * width : nullptr;
     float* dst = out + (size_t)m * width;
+    if (vec) {
+        for (int i = threadIdx.x * 4; i < width; i += blockDim.x * 4) {
+            float4 v = four_of<T>(src + i);
+            v.x *= scale; v.y *= scale; v.z *= scale; v.w *= scale;
+            for (const T* more : {pair, place}) {
+                if (more == nullptr) continue;
+                const float4 w = four_of<T>(more + i);
+                v.x += w.x; v.y += w.y; v.z += w.z; v.w += w.w;
+            }
+            *reinterpret_cast<float4*>(dst + i) = v;
+        }
+        return;
+    }
     for (int i = threadIdx.x; i < width; i += blockDim.x) {
         float v = to_f32<T>(src[i]) * scale;
         if (pair != nullptr) v += to_f32<T>(pair[i]);
@@ -181,14 +203,15 @@ THN_API int thn_embed_rows(float* out, const void* table, const int* tokens, int
     THN_CHECK_ARG(pairs == nullptr || (buckets > 0 && previous != nullptr), "embed_rows: pairs need buckets and the tokens before");
     THN_CHECK_ARG(positions == nullptr || n_positions > 0, "embed_rows: an empty table of positions");
     if (n_rows == 0) return THN_OK;
+    const int vec = width % 4 == 0 && (((uintptr_t)out | (uintptr_t)table | (uintptr_t)pairs | (uintptr_t)positions) & 15) == 0;
     if (dtype == THN_F32)
         thn_launch(embed_rows_kernel<float>, n_rows, 256, 0, stream, out, (const float*)table, tokens, width, n_table_rows, scale,
                    (const float*)pairs, buckets, mul_before, mul_token, previous, (const float*)positions, n_positions, row_slot,
-                   row_pos, cu_seqlens, seq_lens, n_seqs, err);
+                   row_pos, cu_seqlens, seq_lens, n_seqs, vec, err);
     else if (dtype == THN_BF16)
         thn_launch(embed_rows_kernel<__nv_bfloat16>, n_rows, 256, 0, stream, out, (const __nv_bfloat16*)table, tokens, width,
                    n_table_rows, scale, (const __nv_bfloat16*)pairs, buckets, mul_before, mul_token, previous,
-                   (const __nv_bfloat16*)positions, n_positions, row_slot, row_pos, cu_seqlens, seq_lens, n_seqs, err);
+                   (const __nv_bfloat16*)positions, n_positions, row_slot, row_pos, cu_seqlens, seq_lens, n_seqs, vec, err);
     else
         THN_CHECK_ARG(false, "embed_rows: unknown dtype %d", dtype);
     return thn_launch_status("embed_rows");

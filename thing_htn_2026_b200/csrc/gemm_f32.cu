@@ -105,7 +105,7 @@ __global__ void __launch_bounds__(kSkinnyThreads) linear_skinny_kernel(float* __
     const uint4* a = reinterpret_cast<const uint4*>(A);
     const uint4* w = reinterpret_cast<const uint4*>(W);
     const uint4 zero = make_uint4(0, 0, 0, 0);
-    for (int n0 = 0; n0 < N; n0 += 4) {
+    for (int n0 = blockIdx.y * 4; n0 < N; n0 += gridDim.y * 4) {        // four columns at a time
         float acc[ROWS][4];
 #pragma unroll
         for (int r = 0; r < ROWS; ++r)
@@ -148,11 +148,13 @@ THN_API int thn_linear_skinny_bf16(float* C, const void* A, const void* W, int M
     THN_CHECK_ARG(M >= 0 && thn_linear_skinny_supported(N, K), "linear_skinny: bad sizes M=%d N=%d K=%d", M, N, K);
     THN_CHECK_ARG((((uintptr_t)A | (uintptr_t)W) & 15) == 0, "linear_skinny: operands must be 16-byte aligned (M=%d)", M);
     if (M == 0) return THN_OK;
-    if (M >= 1024)      // enough rows to fill the SMs four at a time: the weight's rows are read a quarter as often
+    if (M >= 1024) {    // enough rows to fill the SMs four at a time: the weight's rows are read a quarter as often
         thn_launch(linear_skinny_kernel<4>, (M + 3) / 4, kSkinnyThreads, 0, stream, C, (const __nv_bfloat16*)A,
                    (const __nv_bfloat16*)W, M, N, K / 8);
-    else
-        thn_launch(linear_skinny_kernel<1>, M, kSkinnyThreads, 0, stream, C, (const __nv_bfloat16*)A,
+    } else {            // few rows: the columns are dealt out as well, until there are about two blocks per SM
+        const int groups = (N + 3) / 4, want = (2 * 148 + M - 1) / M;
+        thn_launch(linear_skinny_kernel<1>, dim3(M, groups < want ? groups : want), kSkinnyThreads, 0, stream, C, (const __nv_bfloat16*)A,
                    (const __nv_bfloat16*)W, M, N, K / 8);
+    }
     return thn_launch_status("linear_skinny");
 }

@@ -100,6 +100,97 @@ __global__ void __launch_bounds__(256) latent_assemble_kernel(
     }
 }
 
+// The same for bfloat16 where every part is whole 16-byte pieces (eight entries): a thread takes a piece,
+// or, for half pairs, the two pieces that turn together.
+__device__ __forceinline__ void turn_eight(const uint4& first, const uint4& second, const float* __restrict__ c,
+                                           const float* __restrict__ s, uint4& out_first, uint4& out_second) {
+    const __nv_bfloat162* a2 = reinterpret_cast<const __nv_bfloat162*>(&first);
+    const __nv_bfloat162* b2 = reinterpret_cast<const __nv_bfloat162*>(&second);
+    __nv_bfloat162* x2 = reinterpret_cast<__nv_bfloat162*>(&out_first);
+    __nv_bfloat162* y2 = reinterpret_cast<__nv_bfloat162*>(&out_second);
+#pragma unroll
+    for (int j = 0; j < 4; ++j) {
+        const float2 a = __bfloat1622float2(a2[j]), b = __bfloat1622float2(b2[j]);
+        const float c0 = c[2 * j], c1 = c[2 * j + 1], s0 = s[2 * j], s1 = s[2 * j + 1];
+        x2[j] = __floats2bfloat162_rn(a.x * c0 - b.x * s0, a.y * c1 - b.y * s1);
+        y2[j] = __floats2bfloat162_rn(b.x * c0 + a.x * s0, b.y * c1 + a.y * s1);
+    }
+}
+__device__ __forceinline__ uint4 turn_four_pairs(const uint4& in, const float* __restrict__ c, const float* __restrict__ s) {
+    const __nv_bfloat162* p2 = reinterpret_cast<const __nv_bfloat162*>(&in);
+    uint4 out;
+    __nv_bfloat162* o2 = reinterpret_cast<__nv_bfloat162*>(&out);
+#pragma unroll
+    for (int j = 0; j < 4; ++j) {
+        const float2 v = __bfloat1622float2(p2[j]);
+        o2[j] = __floats2bfloat162_rn(v.x * c[j] - v.y * s[j], v.y * c[j] + v.x * s[j]);
+    }
+    return out;
+}
+
+__global__ void __launch_bounds__(256) latent_assemble_vec_kernel(
+    __nv_bfloat16* __restrict__ q_out, const __nv_bfloat16* __restrict__ q_src, long long q_stride,
+    const __nv_bfloat16* __restrict__ shared_src, long long shared_stride, const __nv_bfloat16* __restrict__ up,
+    const float* __restrict__ cos_tab, const float* __restrict__ sin_tab, int table_len, const int* __restrict__ row_slot,
+    const int* __restrict__ row_pos, PagedKV kv, int n_heads, int plain, int rot, int interleaved, int value_src,
+    int* __restrict__ err) {
+    pdl_launch_dependents();
+    pdl_wait();
+    const int m = blockIdx.x, pos = row_pos[m];
+    const int D = plain + rot, DV = kv.value_dim > 0 ? kv.value_dim : kv.head_dim, half = rot / 2;
+    if (pos >= table_len) {
+        if (threadIdx.x == 0 && err) atomicOr(err, THN_ERR_POSITION_RANGE);
+        return;
+    }
+    const int page = kv.block_table[(size_t)row_slot[m] * kv.bt_stride + pos / kv.page_size];
+    const int in_page = pos % kv.page_size;
+    if (page < 0 && threadIdx.x == 0 && err) atomicOr(err, THN_ERR_PAGE_UNMAPPED);
+    const float* c_row = cos_tab + (size_t)pos * half;
+    const float* s_row = sin_tab + (size_t)pos * half;
+    const __nv_bfloat16* q_row = q_src + (size_t)m * q_stride;
+    const __nv_bfloat16* k_shared = shared_src + (size_t)m * shared_stride;
+    const __nv_bfloat16* up_row = up + (size_t)m * n_heads * (plain + value_src);
+    auto piece = [](const __nv_bfloat16* p) { return *reinterpret_cast<const uint4*>(p); };
+    auto put = [](__nv_bfloat16* p, const uint4& v) { *reinterpret_cast<uint4*>(p) = v; };
+    __nv_bfloat16* cache = page < 0 ? nullptr : (__nv_bfloat16*)kv.base;
+    const long long keys0 = page < 0 ? 0 : kv_offset_sized(kv, page, 0, 0, in_page);
+    const long long values0 = page < 0 ? 0 : kv_offset_sized(kv, page, 1, 0, in_page);
+    const long long key_step = (long long)kv.page_size * D, value_step = (long long)kv.page_size * DV;
+    // work items of a head: plain pieces, turned pieces (pairs of them for half pairs), value pieces
+    const int plain_items = plain / 8, turned_items = interleaved ? rot / 8 : half / 8, value_items = DV / 8;
+    const int per_head = plain_items + turned_items + value_items;
+    for (int item = blockIdx.y * blockDim.x + threadIdx.x; item < n_heads * per_head; item += gridDim.y * blockDim.x) {
+        const int h = item / per_head, i = item - h * per_head;
+        const __nv_bfloat16* q = q_row + (size_t)h * D;
+        __nv_bfloat16* dst = q_out + ((size_t)m * n_heads + h) * D;
+        __nv_bfloat16* key = cache ? cache + keys0 + h * key_step : nullptr;
+        if (i < plain_items) {
+            put(dst + i * 8, piece(q + i * 8));
+            if (key) put(key + i * 8, piece(up_row + (size_t)h * plain + i * 8));
+        } else if (i < plain_items + turned_items) {
+            const int j = (i - plain_items) * 8;
+            if (interleaved) {
+                put(dst + plain + j, turn_four_pairs(piece(q + plain + j), c_row + j / 2, s_row + j / 2));
+                if (key) put(key + plain + j, turn_four_pairs(piece(k_shared + j), c_row + j / 2, s_row + j / 2));
+            } else {
+                uint4 x, y;
+                turn_eight(piece(q + plain + j), piece(q + plain + half + j), c_row + j, s_row + j, x, y);
+                put(dst + plain + j, x);
+                put(dst + plain + half + j, y);
+                if (key) {
+                    turn_eight(piece(k_shared + j), piece(k_shared + half + j), c_row + j, s_row + j, x, y);
+                    put(key + plain + j, x);
+                    put(key + plain + half + j, y);
+                }
+            }
+        } else if (cache) {
+            const int j = (i - plain_items - turned_items) * 8;
+            put(cache + values0 + h * value_step + j,
+                j < value_src ? piece(up_row + (size_t)n_heads * plain + (size_t)h * value_src + j) : make_uint4(0, 0, 0, 0));
+        }
+    }
+}
+
 }  // namespace
 
 // src: rows of the activation type, `rank` entries each, src_stride elements apart; gain float32
@@ -136,6 +227,17 @@ THN_API int thn_latent_assemble(void* q_out, const void* q_src, long long q_stri
     const int D = plain + rot;
     PagedKV kv{kv_base, block_table, bt_stride, n_heads, page_size, D, value_dim == D ? 0 : value_dim};
     if (rot == 0) table_len = 1 << 30;
+    const int turned = interleaved ? rot : rot / 2;
+    if (dtype == THN_BF16 && plain % 8 == 0 && turned % 8 == 0 && value_dim % 8 == 0 && value_src % 8 == 0 && q_stride % 8 == 0 &&
+        shared_stride % 8 == 0 &&
+        (((uintptr_t)q_out | (uintptr_t)q_src | (uintptr_t)shared_src | (uintptr_t)up | (uintptr_t)kv_base) & 15) == 0) {
+        const int items = n_heads * (plain / 8 + turned / 8 + value_dim / 8);
+        const int per_row = n_rows >= 296 ? 1 : (items + 255) / 256;      // few rows: several blocks for each
+        thn_launch(latent_assemble_vec_kernel, dim3(n_rows, per_row), 256, 0, stream, (__nv_bfloat16*)q_out,
+                   (const __nv_bfloat16*)q_src, q_stride, (const __nv_bfloat16*)shared_src, shared_stride, (const __nv_bfloat16*)up,
+                   cos_tab, sin_tab, table_len, row_slot, row_pos, kv, n_heads, plain, rot, interleaved, value_src, err);
+        return thn_launch_status("latent_assemble");
+    }
     if (dtype == THN_F32)
         thn_launch(latent_assemble_kernel<float>, n_rows, 256, 0, stream, (float*)q_out, (const float*)q_src, q_stride,
                    (const float*)shared_src, shared_stride, (const float*)up, cos_tab, sin_tab, table_len, row_slot, row_pos,

@@ -16,16 +16,19 @@
 //
 // Two kernels.  linear_attention_prepare does what is the same for every column, once per entry:
 // silu of q, k and v where asked, the decay with its softplus and exponential, all to float32 rows
-// [row][head][k | q | (decay) | v], the key parts filled up with zeros to a multiple of 32 and the
-// values to a multiple of 16.  linear_attention_kernel is the recurrence.  A column of S (one entry
-// of v and of o) evolves on its own.  It is held by 8 lanes of a warp, lane l keeping the key
-// channels 4l .. 4l + 3, 32 + 4l .. (runs of four, for 16-byte accesses); a token costs each lane
-// its share of multiply-adds and the column three shuffles.  One block per (sequence, head, 16
-// columns) walks the sequence's tokens of the step in order.  The tokens come through shared
-// memory, sixteen at a time (fewer for keys above 128) in two buffers: every thread fetches its
-// 16-byte pieces of the next stage into registers, the block works through the current stage, and
-// then the pieces are stored.  A single-token step is the same two kernels with one token.  A row's
-// result depends on its sequence's own tokens only, in an order fixed by the sizes.
+// [row][head][k | q | (decay) | v], the key parts padded with zeros and the values to a multiple of
+// 16.  linear_attention_kernel is the recurrence, for every mixer that has one of the kinds of
+// linear_attention.cuh.  A column of S (one entry of v and of o) evolves on its own.  16 lanes hold
+// COLS neighbouring columns, lane l the key channels 4l .. 4l + 3, 64 + 4l .. of each (runs of four, for
+// 16-byte accesses), so that a key, query or decay once loaded serves COLS columns.  One block per
+// (sequence, head, 16 columns) walks the sequence's tokens of the step in order.  The tokens come
+// through a ring of buffers in shared memory, filled by asynchronous 16-byte copies.  Eight
+// tokens are worked on together: their state updates follow one another, but their partial sums are
+// reduced over the lanes together, by halving: at every step a lane hands half of its sums to its partner
+// and keeps the other half, so that in the end each lane holds finished sums of its own tokens and columns
+// (15 or 30 shuffles for eight tokens where a butterfly per token takes 32 per column).  What is left of
+// a stage is reduced token by token in the same order of additions.  A row's result depends on
+// its sequence's own tokens only, in an order fixed by the sizes.
 #include <math.h>
 
 #include "linear_attention.cuh"
@@ -34,9 +37,16 @@ namespace {
 
 constexpr int kLanes = kRecurrenceLanes;
 constexpr int kColumns = kRecurrenceColumns;  // columns of S per block
-constexpr int kThreads = kLanes * kColumns;   // 128
-// tokens per stage: fewer for long keys, so that a thread's share of a stage stays in registers
-constexpr int stage_tokens(int per) { return per <= 16 ? 16 : per <= 32 ? 8 : 4; }
+constexpr int kGroup = 8;                     // tokens whose sums are reduced together
+// tokens per buffer, and buffers: fewer tokens for long keys, so that the ring fits
+constexpr int stage_tokens(int per) { return per <= 8 ? 16 : 8; }
+constexpr int kBuffers = 3;
+
+__device__ __forceinline__ void copy16_async(void* smem, const void* gmem) {
+    asm volatile("cp.async.cg.shared.global [%0], [%1], 16;\n" ::"r"((uint32_t)__cvta_generic_to_shared(smem)), "l"(gmem));
+}
+__device__ __forceinline__ void copy_commit() { asm volatile("cp.async.commit_group;\n" ::: "memory"); }
+template <int N> __device__ __forceinline__ void copy_wait() { asm volatile("cp.async.wait_group %0;\n" ::"n"(N) : "memory"); }
 
 // logistic(z)^(1 / tau) = exp(-softplus(-z) / tau), without overflow; in double on the 32-bit path
 template <typename T> __device__ __forceinline__ float logistic_power(float z, float inv_tau) {
@@ -89,153 +99,216 @@ __global__ void linear_attention_prepare_kernel(float* __restrict__ prepared, co
     prepared[e] = v;
 }
 
-// PER: key channels per lane (a multiple of 4); KP = 8 * PER: the padded key size.
-// FETCH: 16-byte pieces per thread and stage, ceil(stage tokens * (parts * KP + 16 + tail) / 4 / 128).
-template <int PER, int KIND, int FETCH>
-__global__ void __launch_bounds__(kThreads) linear_attention_kernel(
+// N sums per lane, to be added over the 16 lanes of a group: the sum at index i ends on the lane
+// whose bits, high to low, are the high bits of i; a lane is left with N / 16 of them (one, if N < 16).
+template <int N>
+__device__ __forceinline__ void reduce_by_halving(float (&part)[N], int lane) {
+    int n = N;
+#pragma unroll
+    for (int off = kLanes / 2; off > 0; off >>= 1) {
+        if (n > 1) {
+            n >>= 1;
+            const bool upper = (lane & off) != 0;
+#pragma unroll
+            for (int i = 0; i < N / 2; ++i) {
+                if (i >= n) break;
+                const float give = upper ? part[i] : part[i + n], keep = upper ? part[i + n] : part[i];
+                part[i] = keep + __shfl_xor_sync(0xffffffffu, give, off);
+            }
+        } else {
+            part[0] += __shfl_xor_sync(0xffffffffu, part[0], off);
+        }
+    }
+}
+
+// PER: key channels per lane (a multiple of 4); KP = 16 * PER: the padded key size.  COLS: columns per lane.
+template <int PER, int COLS, int KIND>
+__global__ void __launch_bounds__(kLanes * kColumns / COLS) linear_attention_kernel(
     float* __restrict__ o, float* __restrict__ state, const float* __restrict__ keys, long long key_stride, int heads_per_unit,
     const float* __restrict__ values, long long value_stride, const float* __restrict__ per_head,
     const int* __restrict__ cu_seqlens, const int* __restrict__ slots, int n_heads, int key_dim, int value_dim, int vp,
     float q_scale) {
     pdl_launch_dependents();
     pdl_wait();
-    constexpr int KP = kLanes * PER, kStage = stage_tokens(PER);
+    constexpr int KP = kLanes * PER, kStage = stage_tokens(PER), kThreads = kLanes * kColumns / COLS;
     constexpr int PARTS = KIND == kChannelDecay || KIND == kBonusRead ? 3 : 2;     // k, q (and the decay) per token
     constexpr int TAIL = KIND >= kBonusRead ? kRecurrenceTail : 0;
-    constexpr int ROW = PARTS * KP + kColumns + TAIL;   // floats of one staged token
+    constexpr int V_AT = PARTS * KP, TAIL_AT = V_AT + kColumns;
+    constexpr int ROW = V_AT + kColumns + TAIL;         // floats of one staged token
     constexpr int PIECES = ROW / 4;
-    extern __shared__ __align__(16) float stage_mem[];  // [2][kStage][ROW]
+    constexpr int SUMS = kGroup * COLS, LEFT = SUMS > kLanes ? SUMS / kLanes : 1;
+    extern __shared__ __align__(16) float stage_mem[];  // [kBuffers][kStage][ROW]
     const int seq = blockIdx.z, head = blockIdx.y;
     const int col0 = blockIdx.x * kColumns;
-    const int column = col0 + threadIdx.x / kLanes;
-    const int lane = threadIdx.x % kLanes;
-    const bool live = column < value_dim;
-    const int col = live ? column : value_dim - 1;     // idle columns mirror the last one and store nothing
+    const int lane = threadIdx.x % kLanes, group = threadIdx.x / kLanes;
+    const int own_col = col0 + group * COLS;           // this lane's first column
     const int row0 = cu_seqlens[seq], row1 = cu_seqlens[seq + 1];
+    if (row0 >= row1) return;
     const int slot = slots[seq];
-    float* S = state + (((size_t)slot * n_heads + head) * value_dim + col) * key_dim;
+    float* S = state + ((size_t)slot * n_heads + head) * (size_t)value_dim * key_dim;
     const int unit = head / heads_per_unit, n_units = n_heads / heads_per_unit;
+    const float* key_src = keys + ((size_t)row0 * n_units + unit) * key_stride;
+    const float* value_src = values + ((size_t)row0 * n_heads + head) * value_stride;
+    const size_t key_step = (size_t)n_units * key_stride, value_step = (size_t)n_heads * value_stride;
+    const int n_tokens = row1 - row0;
 
-    float s[PER];
+    auto issue = [&](int stage) {
+        const int first = stage * kStage, n = min(kStage, n_tokens - first);
+        float* dst = stage_mem + (size_t)(stage % kBuffers) * kStage * ROW;
+        for (int piece = threadIdx.x; piece < n * PIECES; piece += kThreads) {
+            const int t = piece / PIECES, c = (piece - t * PIECES) * 4;
+            const float* src;
+            if (c < V_AT) src = key_src + (size_t)(first + t) * key_step + c;
+            else src = value_src + (size_t)(first + t) * value_step + (TAIL != 0 && c >= TAIL_AT ? vp + (c - TAIL_AT) : col0 + (c - V_AT));
+            copy16_async(dst + piece * 4, src);
+        }
+    };
+    const int n_stages = (n_tokens + kStage - 1) / kStage;
 #pragma unroll
-    for (int i = 0; i < PER; ++i) {
-        const int d = (i / 4) * 32 + lane * 4 + (i & 3);
-        s[i] = d < key_dim ? S[d] : 0.f;
+    for (int i = 0; i < kBuffers - 1; ++i) {
+        if (i < n_stages) issue(i);
+        copy_commit();
+    }
+
+    float s[COLS][PER];
+#pragma unroll
+    for (int c = 0; c < COLS; ++c) {
+        const float* src = S + (size_t)min(own_col + c, value_dim - 1) * key_dim;     // idle columns mirror the last one and store nothing
+#pragma unroll
+        for (int i = 0; i < PER; ++i) {
+            const int d = (i / 4) * (4 * kLanes) + lane * 4 + (i & 3);
+            s[c][i] = d < key_dim ? src[d] : 0.f;
+        }
     }
     const float own = per_head != nullptr ? per_head[head] : 0.f;      // the constant decay, or the skip's factor
 
-    float4 fetched[FETCH];
-    auto fetch = [&](int first_row) {
-        const int n = min(kStage, row1 - first_row);
+    // one token: the sums of its read-out over this lane's channels, and the state behind it
+    auto advance = [&](const float* tok, float (&sums)[COLS]) {
+        float v[COLS];
 #pragma unroll
-        for (int j = 0; j < FETCH; ++j) {
-            const int piece = threadIdx.x + j * kThreads;
-            const int t = piece / PIECES, c = (piece - t * PIECES) * 4;
-            if (t < n) {
-                const float* src;
-                if (c < PARTS * KP) {
-                    src = keys + ((size_t)(first_row + t) * n_units + unit) * key_stride + c;
-                } else {
-                    src = values + ((size_t)(first_row + t) * n_heads + head) * value_stride + (c - PARTS * KP);
-                    src += TAIL != 0 && c >= PARTS * KP + kColumns ? vp - kColumns : col0;
-                }
-                fetched[j] = *reinterpret_cast<const float4*>(src);
+        for (int c = 0; c < COLS; ++c) {
+            v[c] = tok[V_AT + group * COLS + c];
+            sums[c] = 0.f;
+        }
+        float decay = own;
+        if (KIND == kSteppedDecay) {
+            const float2 tail = *reinterpret_cast<const float2*>(tok + TAIL_AT);
+            decay = tail.x;
+#pragma unroll
+            for (int c = 0; c < COLS; ++c) v[c] *= tail.y;
+        }
+#pragma unroll
+        for (int i = 0; i < PER; i += 4) {
+            const int d = (i / 4) * (4 * kLanes) + lane * 4;
+            const float4 k = *reinterpret_cast<const float4*>(tok + d);
+            const float4 q = *reinterpret_cast<const float4*>(tok + KP + d);
+            float4 a = make_float4(decay, decay, decay, decay);
+            if (PARTS == 3) a = *reinterpret_cast<const float4*>(tok + 2 * KP + d);
+#pragma unroll
+            for (int c = 0; c < COLS; ++c) {
+                float* x = s[c] + i;
+                if (KIND == kBonusRead) sums[c] += x[0] * q.x + x[1] * q.y + x[2] * q.z + x[3] * q.w;
+                x[0] = a.x * x[0] + k.x * v[c];
+                x[1] = a.y * x[1] + k.y * v[c];
+                x[2] = a.z * x[2] + k.z * v[c];
+                x[3] = a.w * x[3] + k.w * v[c];
+                if (KIND != kBonusRead) sums[c] += x[0] * q.x + x[1] * q.y + x[2] * q.z + x[3] * q.w;
             }
         }
     };
-    auto publish = [&](int buf, int n) {
-        float* dst = stage_mem + (size_t)buf * kStage * ROW;
-#pragma unroll
-        for (int j = 0; j < FETCH; ++j) {
-            const int piece = threadIdx.x + j * kThreads;
-            if (piece / PIECES < n) *reinterpret_cast<float4*>(dst + piece * 4) = fetched[j];
-        }
+    // the finished sum of column c of this lane's group, for the stage's token at tok, row `row`
+    auto store = [&](const float* tok, int row, int c, float sum) {
+        const int column = own_col + c;
+        if (column >= value_dim) return;
+        float y = sum * q_scale;
+        if (KIND == kBonusRead) y += tok[TAIL_AT] * tok[V_AT + group * COLS + c];
+        if (KIND == kSteppedDecay) y += own * tok[V_AT + group * COLS + c];
+        o[((size_t)row * n_heads + head) * value_dim + column] = y;
     };
 
-    if (row0 < row1) {
-        fetch(row0);
-        publish(0, min(kStage, row1 - row0));
-    }
-    __syncthreads();
-    const int v_at = PARTS * KP + threadIdx.x / kLanes;
-    for (int first = row0, buf = 0; first < row1; first += kStage, buf ^= 1) {
-        const bool more = first + kStage < row1;
-        if (more) fetch(first + kStage);
-        // the loads stay here, ahead of the stage's work: sunk to where their values are stored, each
-        // would wait for memory in its turn
-        asm volatile("" ::: "memory");
-        const float* src = stage_mem + (size_t)buf * kStage * ROW;
-        const int n = min(kStage, row1 - first);
-        // (unrolled: only the state's multiply-adds link one token to the next; the loads and the
-        // shuffles of two tokens then overlap)
-#pragma unroll 2
-        for (int t = 0; t < n; ++t) {
-            const float* tok = src + t * ROW;
-            const float shown = tok[v_at];
-            float v = shown, decay = own, bonus = 0.f;
-            if (KIND == kBonusRead) bonus = tok[PARTS * KP + kColumns];
-            if (KIND == kSteppedDecay) {
-                decay = tok[PARTS * KP + kColumns];
-                v = shown * tok[PARTS * KP + kColumns + 1];
-            }
-            float part = 0.f;
+    for (int stage = 0; stage < n_stages; ++stage) {
+        copy_wait<kBuffers - 2>();
+        __syncthreads();                     // this stage has landed; the buffer of the one before it is free again
+        if (stage + kBuffers - 1 < n_stages) issue(stage + kBuffers - 1);
+        copy_commit();
+        const float* src = stage_mem + (size_t)(stage % kBuffers) * kStage * ROW;
+        const int first = stage * kStage, n = min(kStage, n_tokens - first);
+        int t0 = 0;
+#pragma unroll 1
+        for (; t0 + kGroup <= n; t0 += kGroup) {
+            float part[SUMS];
 #pragma unroll
-            for (int i = 0; i < PER; i += 4) {
-                const int d = (i / 4) * 32 + lane * 4;
-                const float4 k = *reinterpret_cast<const float4*>(tok + d);
-                const float4 q = *reinterpret_cast<const float4*>(tok + KP + d);
-                float4 a = make_float4(decay, decay, decay, decay);
-                if (PARTS == 3) a = *reinterpret_cast<const float4*>(tok + 2 * KP + d);
-                if (KIND == kBonusRead) part += s[i] * q.x + s[i + 1] * q.y + s[i + 2] * q.z + s[i + 3] * q.w;
-                s[i] = a.x * s[i] + k.x * v;
-                s[i + 1] = a.y * s[i + 1] + k.y * v;
-                s[i + 2] = a.z * s[i + 2] + k.z * v;
-                s[i + 3] = a.w * s[i + 3] + k.w * v;
-                if (KIND != kBonusRead) part += s[i] * q.x + s[i + 1] * q.y + s[i + 2] * q.z + s[i + 3] * q.w;
-            }
+            for (int t = 0; t < kGroup; ++t) {
+                float sums[COLS];
+                advance(src + (t0 + t) * ROW, sums);
 #pragma unroll
-            for (int off = kLanes / 2; off > 0; off >>= 1) part += __shfl_xor_sync(0xffffffffu, part, off);
-            if (lane == 0 && live) {
-                float y = part * q_scale;
-                if (KIND == kBonusRead) y += bonus * shown;
-                if (KIND == kSteppedDecay) y += own * shown;
-                o[((size_t)(first + t) * n_heads + head) * value_dim + col] = y;
+                for (int c = 0; c < COLS; ++c) part[t * COLS + c] = sums[c];
+            }
+            reduce_by_halving<SUMS>(part, lane);
+            const int index = SUMS >= kLanes ? lane * LEFT : lane / (kLanes / SUMS);
+            if (SUMS >= kLanes || lane % (kLanes / (SUMS < kLanes ? SUMS : 1)) == 0) {
+#pragma unroll
+                for (int j = 0; j < LEFT; ++j) {
+                    const int t = t0 + (index + j) / COLS;
+                    store(src + t * ROW, row0 + first + t, (index + j) % COLS, part[j]);
+                }
             }
         }
-        if (more) publish(buf ^ 1, min(kStage, row1 - first - kStage));
-        __syncthreads();
+#pragma unroll 1
+        for (; t0 < n; ++t0) {
+            float sums[COLS];
+            advance(src + t0 * ROW, sums);
+#pragma unroll
+            for (int off = kLanes / 2; off > 0; off >>= 1)
+#pragma unroll
+                for (int c = 0; c < COLS; ++c) sums[c] += __shfl_xor_sync(0xffffffffu, sums[c], off);
+            if (lane == 0) {
+#pragma unroll
+                for (int c = 0; c < COLS; ++c) store(src + t0 * ROW, row0 + first + t0, c, sums[c]);
+            }
+        }
     }
-    if (live && row0 < row1) {
+#pragma unroll
+    for (int c = 0; c < COLS; ++c) {
+        if (own_col + c >= value_dim) break;
+        float* dst = S + (size_t)(own_col + c) * key_dim;
 #pragma unroll
         for (int i = 0; i < PER; ++i) {
-            const int d = (i / 4) * 32 + lane * 4 + (i & 3);
-            if (d < key_dim) S[d] = s[i];
+            const int d = (i / 4) * (4 * kLanes) + lane * 4 + (i & 3);
+            if (d < key_dim) dst[d] = s[c][i];
         }
     }
 }
 
-template <int PER, int KIND>
+template <int PER, int COLS, int KIND>
 void launch_one(const RecurrenceArgs& a, cudaStream_t stream) {
     constexpr int KP = kLanes * PER, kStage = stage_tokens(PER);
     constexpr int ROW = (KIND == kChannelDecay || KIND == kBonusRead ? 3 : 2) * KP + kColumns + (KIND >= kBonusRead ? kRecurrenceTail : 0);
-    constexpr int FETCH = (kStage * ROW / 4 + kThreads - 1) / kThreads;
-    const size_t smem = 2 * (size_t)kStage * ROW * sizeof(float);
+    const size_t smem = kBuffers * (size_t)kStage * ROW * sizeof(float);
     const dim3 grid((a.value_dim + kColumns - 1) / kColumns, a.n_heads, a.n_seqs);
-    auto kernel = linear_attention_kernel<PER, KIND, FETCH>;
+    auto kernel = linear_attention_kernel<PER, COLS, KIND>;
     if (smem > 48 * 1024) cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-    thn_launch_ordered(kernel, grid, kThreads, smem, stream, a.o, a.state, a.keys, a.key_stride, a.n_heads / a.key_units, a.values,
-                       a.value_stride, a.per_head, a.cu_seqlens, a.slots, a.n_heads, a.key_dim, a.value_dim,
+    thn_launch_ordered(kernel, grid, kLanes * kColumns / COLS, smem, stream, a.o, a.state, a.keys, a.key_stride, a.n_heads / a.key_units,
+                       a.values, a.value_stride, a.per_head, a.cu_seqlens, a.slots, a.n_heads, a.key_dim, a.value_dim,
                        padded_values(a.value_dim), a.q_scale);
+}
+
+int g_columns = 0;      // columns per lane for keys up to 128: 1, 2, 4, or 0: the default
+
+template <int PER, int KIND>
+void launch_columns(const RecurrenceArgs& a, int columns, cudaStream_t stream) {
+    if (columns == 4) launch_one<PER, 4, KIND>(a, stream);
+    else if (columns == 2) launch_one<PER, 2, KIND>(a, stream);
+    else launch_one<PER, 1, KIND>(a, stream);
 }
 
 template <int KIND>
 void launch_kind(const RecurrenceArgs& a, cudaStream_t stream) {
     switch (recurrence_per_lane(a.key_dim)) {
-        case 4: return launch_one<4, KIND>(a, stream);
-        case 8: return launch_one<8, KIND>(a, stream);
-        case 16: return launch_one<16, KIND>(a, stream);
-        case 32: return launch_one<32, KIND>(a, stream);
-        default: return launch_one<64, KIND>(a, stream);
+        case 4: return launch_columns<4, KIND>(a, g_columns ? g_columns : 2, stream);
+        case 8: return launch_columns<8, KIND>(a, g_columns ? g_columns : 2, stream);
+        case 16: return launch_one<16, 2, KIND>(a, stream);
+        default: return launch_one<32, 1, KIND>(a, stream);
     }
 }
 
@@ -255,6 +328,9 @@ int launch(float* o, float* state, float* prepared, const void* proj, int proj_w
 }
 
 }  // namespace
+
+// How many columns of S a lane holds, for keys up to 128 (tests and measurement): 1, 2, 4, or 0: the default.
+THN_API void thn_set_recurrence_columns(int columns) { g_columns = columns == 1 || columns == 2 || columns == 4 ? columns : 0; }
 
 int launch_recurrence(int kind, const RecurrenceArgs& args, cudaStream_t stream) {
     THN_CHECK_ARG(args.key_units > 0 && args.n_heads % args.key_units == 0, "recurrence: %d heads over %d units of keys",

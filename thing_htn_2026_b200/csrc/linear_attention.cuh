@@ -19,15 +19,12 @@
 
 enum RecurrenceKind { kConstantDecay = 0, kChannelDecay = 1, kBonusRead = 2, kSteppedDecay = 3 };
 
-constexpr int kRecurrenceLanes = 8;        // lanes that hold a column of S
+constexpr int kRecurrenceLanes = 16;       // lanes that hold a column of S
 constexpr int kRecurrenceColumns = 16;     // columns of S per block
 constexpr int kRecurrenceTail = 4;
 
 // key channels per lane: runs of four
-inline int recurrence_per_lane(int key_dim) {
-    const int per = (key_dim + 31) / 32 * 4;
-    return per <= 4 ? 4 : per <= 8 ? 8 : per <= 16 ? 16 : per <= 32 ? 32 : 64;
-}
+inline int recurrence_per_lane(int key_dim) { return key_dim <= 64 ? 4 : key_dim <= 128 ? 8 : key_dim <= 256 ? 16 : 32; }
 inline int padded_keys(int key_dim) { return kRecurrenceLanes * recurrence_per_lane(key_dim); }
 inline int padded_values(int value_dim) { return (value_dim + kRecurrenceColumns - 1) / kRecurrenceColumns * kRecurrenceColumns; }
 inline int key_parts(int kind) { return kind == kChannelDecay || kind == kBonusRead ? 3 : 2; }

@@ -339,7 +339,7 @@ __global__ void __launch_bounds__(256) gated_row_norm_kernel(T* __restrict__ out
 __global__ void gated_head_norm_bf16_vec_kernel(__nv_bfloat16* __restrict__ out, const float* __restrict__ o,
                                                 const __nv_bfloat16* __restrict__ gate, long long gate_stride,
                                                 const float* __restrict__ w, float eps, long long n_units, int n_heads,
-                                                int size) {
+                                                int size, int w_stride) {
     pdl_launch_dependents();
     pdl_wait();
     const int lane = threadIdx.x & 31;
@@ -349,6 +349,7 @@ __global__ void gated_head_norm_bf16_vec_kernel(__nv_bfloat16* __restrict__ out,
     const int head = (int)(unit - m * n_heads);
     const float* src = o + unit * size;
     const __nv_bfloat16* g = gate + m * gate_stride + (long long)head * size;
+    const float* wh = w + (size_t)head * w_stride;
     float4 first = make_float4(0, 0, 0, 0);          // the first chunk stays in registers (sizes up to 128: the only one)
     float ss = 0.f;
     for (int i = lane * 4; i < size; i += 128) {
@@ -360,7 +361,7 @@ __global__ void gated_head_norm_bf16_vec_kernel(__nv_bfloat16* __restrict__ out,
     const float rstd = 1.0f / sqrtf(ss / (float)size + eps);
     for (int i = lane * 4; i < size; i += 128) {
         const float4 v = i < 128 ? first : *reinterpret_cast<const float4*>(src + i);
-        const float4 gw = *reinterpret_cast<const float4*>(w + i);
+        const float4 gw = *reinterpret_cast<const float4*>(wh + i);
         const uint2 gz = *reinterpret_cast<const uint2*>(g + i);
         const float2 z0 = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&gz.x));
         const float2 z1 = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&gz.y));
@@ -419,11 +420,11 @@ THN_API int thn_gated_head_norm(void* out, const float* o, const void* gate, lon
     const int w_stride = w_per_head ? size : 0;
     if (out_stride <= 0) out_stride = (long long)n_heads * size;
     THN_CHECK_ARG(out_stride >= (long long)n_heads * size, "gated_head_norm: output rows %lld apart are too short", out_stride);
-    if (dtype == THN_BF16 && !w_per_head && gate_kind == 0 && size % 4 == 0 && gate_stride % 4 == 0 && scale == 1.0f &&
+    if (dtype == THN_BF16 && gate_kind == 0 && size % 4 == 0 && gate_stride % 4 == 0 && scale == 1.0f &&
         out_stride == (long long)n_heads * size &&
         ((((uintptr_t)o | (uintptr_t)w) & 15) | (((uintptr_t)gate | (uintptr_t)out) & 7)) == 0) {
         thn_launch(gated_head_norm_bf16_vec_kernel, blocks, warps * 32, 0, stream, (__nv_bfloat16*)out, o,
-                   (const __nv_bfloat16*)gate, gate_stride, w, eps, units, n_heads, size);
+                   (const __nv_bfloat16*)gate, gate_stride, w, eps, units, n_heads, size, w_stride);
         return thn_launch_status("gated_head_norm");
     }
     if (n_heads == 1 && size >= 512 && (dtype == THN_F32 || dtype == THN_BF16)) {

@@ -144,6 +144,7 @@ __global__ void __launch_bounds__(kPrepareThreads) state_space_prepare_kernel(
 }
 
 constexpr int kDecodeThreads = 256;
+constexpr int kDecodeLanes = 8;            // lanes that share a column of S
 
 // Shared memory: B, C [n_state] each, x [vdim].
 template <typename T>
@@ -185,8 +186,8 @@ __global__ void __launch_bounds__(kDecodeThreads) state_space_decode_kernel(
     const float decay = exp_of<T>(-rate[head] * t), d_skip = skip[head];
     __syncthreads();
     float* S = state + ((size_t)slot * shape.n_heads + head) * V * N;
-    const int lane = threadIdx.x % kRecurrenceLanes, column = threadIdx.x / kRecurrenceLanes;
-    constexpr int kGroups = kDecodeThreads / kRecurrenceLanes;
+    const int lane = threadIdx.x % kDecodeLanes, column = threadIdx.x / kDecodeLanes;
+    constexpr int kGroups = kDecodeThreads / kDecodeLanes;
     const bool vec = N % 4 == 0;
     for (int e0 = 0; e0 < V; e0 += kGroups) {
         const int e = e0 + column;
@@ -195,7 +196,7 @@ __global__ void __launch_bounds__(kDecodeThreads) state_space_decode_kernel(
             float* col = S + (size_t)e * N;
             const float tx = t * xs[e];
             if (vec) {
-                for (int d = lane * 4; d < N; d += kRecurrenceLanes * 4) {
+                for (int d = lane * 4; d < N; d += kDecodeLanes * 4) {
                     float4 s = *reinterpret_cast<const float4*>(col + d);
                     const float4 b = *reinterpret_cast<const float4*>(bs + d), c = *reinterpret_cast<const float4*>(cs + d);
                     s.x = decay * s.x + b.x * tx;
@@ -206,7 +207,7 @@ __global__ void __launch_bounds__(kDecodeThreads) state_space_decode_kernel(
                     *reinterpret_cast<float4*>(col + d) = s;
                 }
             } else {
-                for (int d = lane; d < N; d += kRecurrenceLanes) {
+                for (int d = lane; d < N; d += kDecodeLanes) {
                     const float s = decay * col[d] + bs[d] * tx;
                     part += s * cs[d];
                     col[d] = s;
@@ -214,12 +215,12 @@ __global__ void __launch_bounds__(kDecodeThreads) state_space_decode_kernel(
             }
         }
 #pragma unroll
-        for (int off = kRecurrenceLanes / 2; off > 0; off >>= 1) part += __shfl_xor_sync(0xffffffffu, part, off);
+        for (int off = kDecodeLanes / 2; off > 0; off >>= 1) part += __shfl_xor_sync(0xffffffffu, part, off);
         if (lane == 0 && e < V) y[((size_t)row * shape.n_heads + head) * V + e] = part + d_skip * xs[e];
     }
 }
 
-// One block per (row, part).  The gated entries are computed twice, once for the sum of squares and
+// One block per (row, part), with as many threads as the part has pieces of four entries, up to 256.  The gated entries are computed twice, once for the sum of squares and
 // once for the result; the second reading comes from the caches.
 template <typename T>
 __global__ void __launch_bounds__(256) gated_group_norm_kernel(T* __restrict__ out, const float* __restrict__ y,
@@ -236,18 +237,18 @@ __global__ void __launch_bounds__(256) gated_group_norm_kernel(T* __restrict__ o
     T* dst = out + base;
     float ss = 0.f;
     if (vec) {
-        constexpr int kKept = 4;                    // what fits stays in registers (parts up to 4096 entries)
+        constexpr int kKept = 4;                    // what fits stays in registers (parts up to sixteen entries a thread)
         float4 kept[kKept];
 #pragma unroll
         for (int j = 0; j < kKept; ++j) {
-            const int i = (j * 256 + threadIdx.x) * 4;
+            const int i = (j * (int)blockDim.x + (int)threadIdx.x) * 4;
             if (i < size) {
                 const float4 v = *reinterpret_cast<const float4*>(src + i), z = load_four<T>(g + i);
                 kept[j] = make_float4(v.x * silu_of<T>(z.x), v.y * silu_of<T>(z.y), v.z * silu_of<T>(z.z), v.w * silu_of<T>(z.w));
                 ss += kept[j].x * kept[j].x + kept[j].y * kept[j].y + kept[j].z * kept[j].z + kept[j].w * kept[j].w;
             }
         }
-        for (int i = (kKept * 256 + threadIdx.x) * 4; i < size; i += 1024) {
+        for (int i = (kKept * (int)blockDim.x + (int)threadIdx.x) * 4; i < size; i += (int)blockDim.x * 4) {
             const float4 v = *reinterpret_cast<const float4*>(src + i), z = load_four<T>(g + i);
             const float a = v.x * silu_of<T>(z.x), b = v.y * silu_of<T>(z.y), c = v.z * silu_of<T>(z.z), d = v.w * silu_of<T>(z.w);
             ss += a * a + b * b + c * c + d * d;
@@ -266,21 +267,21 @@ __global__ void __launch_bounds__(256) gated_group_norm_kernel(T* __restrict__ o
         };
 #pragma unroll
         for (int j = 0; j < kKept; ++j) {
-            const int i = (j * 256 + threadIdx.x) * 4;
+            const int i = (j * (int)blockDim.x + (int)threadIdx.x) * 4;
             if (i < size) store(i, kept[j]);
         }
-        for (int i = (kKept * 256 + threadIdx.x) * 4; i < size; i += 1024) {
+        for (int i = (kKept * (int)blockDim.x + (int)threadIdx.x) * 4; i < size; i += (int)blockDim.x * 4) {
             const float4 v = *reinterpret_cast<const float4*>(src + i), z = load_four<T>(g + i);
             store(i, make_float4(v.x * silu_of<T>(z.x), v.y * silu_of<T>(z.y), v.z * silu_of<T>(z.z), v.w * silu_of<T>(z.w)));
         }
         return;
     }
-    for (int i = threadIdx.x; i < size; i += 256) {
+    for (int i = threadIdx.x; i < size; i += blockDim.x) {
         const float v = src[i] * silu_of<T>(to_f32<T>(g[i]));
         ss += v * v;
     }
     const float rstd = 1.0f / sqrtf(block_sum(ss, scratch) / (float)size + eps);
-    for (int i = threadIdx.x; i < size; i += 256) dst[i] = from_f32<T>(src[i] * silu_of<T>(to_f32<T>(g[i])) * rstd * w[i]);
+    for (int i = threadIdx.x; i < size; i += blockDim.x) dst[i] = from_f32<T>(src[i] * silu_of<T>(to_f32<T>(g[i])) * rstd * w[i]);
 }
 
 int check_shape(const char* what, const SpaceShape& s, int proj_width, int offset) {
@@ -388,11 +389,12 @@ THN_API int thn_gated_group_norm(void* out, const float* y, const void* gate, lo
     const int vec = size % 4 == 0 && gate_stride % 4 == 0 && (((uintptr_t)y | (uintptr_t)gain) & 15) == 0 &&
                     (((uintptr_t)gate | (uintptr_t)out) & (4 * element - 1)) == 0;
     const dim3 grid(rows, parts);
+    const int threads = size >= 1024 ? 256 : (size / 4 + 31) / 32 * 32 < 32 ? 32 : (size / 4 + 31) / 32 * 32;
     if (dtype == THN_F32)
-        thn_launch(gated_group_norm_kernel<float>, grid, 256, 0, stream, (float*)out, y, (const float*)gate, gate_stride, gain, eps,
+        thn_launch(gated_group_norm_kernel<float>, grid, threads, 0, stream, (float*)out, y, (const float*)gate, gate_stride, gain, eps,
                    width, size, vec);
     else if (dtype == THN_BF16)
-        thn_launch(gated_group_norm_kernel<__nv_bfloat16>, grid, 256, 0, stream, (__nv_bfloat16*)out, y, (const __nv_bfloat16*)gate,
+        thn_launch(gated_group_norm_kernel<__nv_bfloat16>, grid, threads, 0, stream, (__nv_bfloat16*)out, y, (const __nv_bfloat16*)gate,
                    gate_stride, gain, eps, width, size, vec);
     else
         THN_CHECK_ARG(false, "gated_group_norm: unknown dtype %d", dtype);

@@ -154,6 +154,7 @@ __global__ void __launch_bounds__(kPrepareWarps * 32) wkv_prepare_kernel(
 }
 
 constexpr int kDecodeThreads = 256;
+constexpr int kDecodeLanes = 8;            // lanes that share a column of S
 
 // Shared memory: r, k, v, w [dim] each, tanh'd low-rank input [rank], the read-out [dim].
 template <typename T>
@@ -195,8 +196,8 @@ __global__ void __launch_bounds__(kDecodeThreads) wkv_decode_kernel(
     }
     __syncthreads();
     float* S = state + ((size_t)row_slot[row] * n_heads + head) * dim * dim;
-    const int lane = threadIdx.x % kRecurrenceLanes, group = threadIdx.x / kRecurrenceLanes;
-    constexpr int kGroups = kDecodeThreads / kRecurrenceLanes;
+    const int lane = threadIdx.x % kDecodeLanes, group = threadIdx.x / kDecodeLanes;
+    constexpr int kGroups = kDecodeThreads / kDecodeLanes;
     const bool vec = dim % 4 == 0;
     for (int e0 = 0; e0 < dim; e0 += kGroups) {
         const int e = e0 + group;
@@ -205,7 +206,7 @@ __global__ void __launch_bounds__(kDecodeThreads) wkv_decode_kernel(
             float* col = S + (size_t)e * dim;
             const float ve = vs[e];
             if (vec) {
-                for (int d = lane * 4; d < dim; d += kRecurrenceLanes * 4) {
+                for (int d = lane * 4; d < dim; d += kDecodeLanes * 4) {
                     float4 s = *reinterpret_cast<const float4*>(col + d);
                     const float4 rd = *reinterpret_cast<const float4*>(rs + d), kd = *reinterpret_cast<const float4*>(ks + d);
                     const float4 wd = *reinterpret_cast<const float4*>(ws + d);
@@ -217,7 +218,7 @@ __global__ void __launch_bounds__(kDecodeThreads) wkv_decode_kernel(
                     *reinterpret_cast<float4*>(col + d) = s;
                 }
             } else {
-                for (int d = lane; d < dim; d += kRecurrenceLanes) {
+                for (int d = lane; d < dim; d += kDecodeLanes) {
                     const float s = col[d];
                     part += s * rs[d];
                     col[d] = ws[d] * s + ks[d] * ve;
@@ -225,7 +226,7 @@ __global__ void __launch_bounds__(kDecodeThreads) wkv_decode_kernel(
             }
         }
 #pragma unroll
-        for (int off = kRecurrenceLanes / 2; off > 0; off >>= 1) part += __shfl_xor_sync(0xffffffffu, part, off);
+        for (int off = kDecodeLanes / 2; off > 0; off >>= 1) part += __shfl_xor_sync(0xffffffffu, part, off);
         if (lane == 0 && e < dim) os[e] = part + share * vs[e];
     }
     __syncthreads();

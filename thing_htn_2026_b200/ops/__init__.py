@@ -189,6 +189,8 @@ def lib():
         loaded.thn_attention_decode_scratch_floats.restype = c_longlong
         loaded.thn_linear_attention_scratch_floats.argtypes = [c_int, c_int, c_int, c_int, c_int]
         loaded.thn_linear_attention_scratch_floats.restype = c_longlong
+        loaded.thn_set_recurrence_columns.argtypes = [c_int]
+        loaded.thn_set_recurrence_columns.restype = None
         loaded.thn_wkv_scratch_floats.argtypes = [c_int, c_int, c_int]
         loaded.thn_wkv_scratch_floats.restype = c_longlong
         loaded.thn_state_space_scratch_floats.argtypes = [c_int, c_int, c_int, c_int, c_int]
@@ -722,12 +724,19 @@ def linear_swiglu(x: torch.Tensor, w_gate_up: torch.Tensor, err: Optional[torch.
     return swiglu(linear(x, w_gate_up, err=err))
 
 
+# The warp-per-row product re-reads its weight for every few rows: with many rows and more than a few
+# columns the vendor library's tensor-core product is faster (2,048 rows, 64 columns over 2,048: 62 us
+# for the former on B200).
+SKINNY_MAX_ROWS = 256
+SKINNY_ANY_ROWS_COLUMNS = 16
+
+
 def linear(x: torch.Tensor, weight: torch.Tensor, out_dtype: Optional[torch.dtype] = None,
            err: Optional[torch.Tensor] = None, bias: Optional[torch.Tensor] = None) -> torch.Tensor:
     """x [M, K] @ weight[N, K]^T.  float32: this library's FFMA kernel.  bfloat16 with few
     rows and a deep reduction or a tall weight: this library's weight-streaming kernel
     (``err``: the step's device error word for its bounded waits).  bfloat16 with a float32 result
-    of at most 64 columns (a router, a gate): this library's warp-per-row kernel.  bfloat16 otherwise: the
+    of at most 64 columns (a router, a gate; with many rows of at most 16): this library's warp-per-row kernel.  bfloat16 otherwise: the
     vendor library's tensor-core product with float32 accumulation (the reference's choice,
     engine/engine.py:341-350).  ``out_dtype=torch.float32`` keeps the accumulator's
     precision (used for logits).  ``bias`` (of the activation type, ``[N]``) is added to every row:
@@ -759,6 +768,7 @@ def linear(x: torch.Tensor, weight: torch.Tensor, out_dtype: Optional[torch.dtyp
     if x.dtype != torch.bfloat16:
         raise KernelError(f"linear: dtype {x.dtype} is not supported")
     if (out_dtype == torch.float32 and lib().thn_linear_skinny_supported(weight.shape[0], x.shape[1])
+            and (x.shape[0] < SKINNY_MAX_ROWS or weight.shape[0] <= SKINNY_ANY_ROWS_COLUMNS)
             and (x.data_ptr() | weight.data_ptr()) % 16 == 0):
         # a router or a gate: a few float32 outputs per row, on this library's warp-per-row kernel
         out = torch.empty((x.shape[0], weight.shape[0]), dtype=torch.float32, device=x.device)
@@ -1504,6 +1514,12 @@ def hyper_norm(streams: Optional[torch.Tensor], n_streams: int, dtype: torch.dty
 # ------------------------------------------------------------------ linear attention, selective scan
 
 
+def set_recurrence_columns(columns: int = 0) -> None:
+    """How many columns of the state a lane of the shared recurrence kernel holds, for keys up to 128
+    (tests and measurement): 1, 2, 4, or 0: the default."""
+    lib().thn_set_recurrence_columns(int(columns))
+
+
 def linear_attention(proj: torch.Tensor, offsets: Tuple[int, int, int], state: torch.Tensor, rows: StepRows,
                      n_heads: int, key_dim: int, value_dim: int, *, decay: Optional[torch.Tensor] = None,
                      gate: Optional[torch.Tensor] = None, gate_bias: Optional[torch.Tensor] = None, tau: float = 1.0,
@@ -1839,5 +1855,5 @@ def gather_i32(src: torch.Tensor, index: torch.Tensor, out: Optional[torch.Tenso
 __all__ = [
     "KernelError", "KernelLibraryError", "KVView", "RotaryTables", "RowTiles", "StepRows", "row_tiles_of", "prompt_attention_tile", "linear_stream", "linear_swiglu", "linear_tcgen05", "add_rmsnorm", "advance",
     "ROW_TILE", "attention", "attention_decode_bf16", "attention_generic", "attention_prefill_bf16", "attention_prefill_tcgen05", "decode_splits", "choose_tokens", "gather_i32", "gather_rows", "lib", "linear", "new_error_word",
-    "qk_norm_rope_cache", "qk_prepare", "Gain", "STREAM_AS_IS", "residual_norm", "gather_rows_scaled", "logistic_gate", "latent_norm", "latent_assemble", "mlstm", "mlstm_column_blocks", "set_mlstm_kernel", "Routing", "moe_route", "routed_gelu", "gated_head_norm", "clamped_glu", "routed_clamped_glu", "polynorm", "scale_", "ScoreShape", "PLAIN_SCORES", "DeltaShape", "delta_rule", "qkv_attention", "raise_on_device_error", "rmsnorm", "StreamNumbers", "hyper_norm", "linear_attention", "causal_conv", "conv_ring_update", "selective_scan", "PairTable", "embed_rows", "squared_relu", "linear_batched", "token_shift", "tanh_rows", "wkv", "wkv_decode", "StateSpace", "state_space", "gated_group_norm", "rotate_gate", "rope_table", "scatter_i32", "step_rows", "swiglu",
+    "qk_norm_rope_cache", "qk_prepare", "Gain", "STREAM_AS_IS", "residual_norm", "gather_rows_scaled", "logistic_gate", "latent_norm", "latent_assemble", "mlstm", "mlstm_column_blocks", "set_mlstm_kernel", "Routing", "moe_route", "routed_gelu", "gated_head_norm", "clamped_glu", "routed_clamped_glu", "polynorm", "scale_", "ScoreShape", "PLAIN_SCORES", "DeltaShape", "delta_rule", "qkv_attention", "raise_on_device_error", "rmsnorm", "StreamNumbers", "hyper_norm", "linear_attention", "set_recurrence_columns", "causal_conv", "conv_ring_update", "selective_scan", "PairTable", "embed_rows", "squared_relu", "linear_batched", "token_shift", "tanh_rows", "wkv", "wkv_decode", "StateSpace", "state_space", "gated_group_norm", "rotate_gate", "rope_table", "scatter_i32", "step_rows", "swiglu",
 ]
