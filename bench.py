@@ -1436,7 +1436,7 @@ def futepel_kernel_table(torch, fut, peak, batch, context):
         row(f"{tag}: linear_batched (r, k, v, gate)", lambda: ops.linear_batched(blends[:4], w_wide),
             like=f"{tag}: linear (one product of the same size)", **prod)
         row(f"{tag}: linear (one product of the same size)", lambda: ops.linear(d16, w_one, err=err), **prod)
-        row(f"{tag}: linear (decay, first)", lambda: ops.linear(blends[4], w1, out_dtype=torch.float32, err=err),
+        row(f"{tag}: linear (decay, first)", lambda: ops.linear(blends[4], w1, out_dtype=torch.float32, err=err, rows_alone=False),
             flops=2.0 * m * W * rank, nbytes=W * rank * 2 + m * (W * 2 + rank * 4))
         planes, low = (rnd(4, m, h * d) * 0.5).to(bf), rnd(m, rank)
         lin = rnd(m, Hg * 4 * dg).to(bf) * 0.5

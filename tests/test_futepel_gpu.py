@@ -547,6 +547,40 @@ def test_state_space_keeps_a_far_input_by_its_decay(dtype, heads, groups, e, n, 
         seqs.cache.close([slot])
 
 
+@pytest.mark.parametrize("columns", [1, 2, 4])
+@pytest.mark.parametrize("heads, d", [(3, 24), (2, 64), (2, 100), (1, 128)])
+def test_every_variant_of_the_recurrence(columns, heads, d):
+    """The shared recurrence with 1, 2 and 4 columns of the state in a lane, over prompts of 1, 7, 37 and
+    100 tokens side by side (whole stages, groups of eight and what is left), against token by token in
+    double, with the states that they leave."""
+    from thing_htn_2026_b200 import ops
+    from thing_htn_2026_b200.cache.sequence_cache import StateSpec
+    counts = [1, 37, 100, 7]
+    n = sum(counts)
+    planes, z = rand((3, n, heads * d), 1), rand((n, heads * d), 2)
+    w0, u, S0 = rand((heads * d,), 3).sub(3.0), rand((heads, d), 4), rand((len(counts), heads, d, d), 5, 0.3)
+    seqs = Sequences([StateSpec((heads, d, d))], "float32", n_slots=5)
+    slots = seqs.cache.open(4)
+    seqs.cache.state_view(0)[torch.tensor(slots)] = S0.to(DEV)
+    rows = seqs.rows(slots, counts)
+    ops.set_recurrence_columns(columns)
+    try:
+        got = ops.wkv(planes.to(DEV), z.to(DEV), w0.to(DEV), u.to(DEV), seqs.cache.state_view(0), rows, heads, d).cpu().double()
+    finally:
+        ops.set_recurrence_columns(0)
+    left = seqs.cache.state_view(0)[torch.tensor(slots)].cpu().double()
+    r, k, v = (p.double().view(n, heads, d) for p in planes)
+    w = torch.exp(-torch.exp(z.double() + w0.double())).view(n, heads, d)
+    for i, (lo, hi) in enumerate(zip(seqs.cu[:-1], seqs.cu[1:])):
+        S = S0[i].double()                                          # [head, value, key]
+        for t in range(lo, hi):
+            kv = v[t][:, :, None] * k[t][:, None, :]
+            want = ((S + u.double()[:, None, :] * kv) * r[t][:, None, :]).sum(-1)
+            assert (got[t] - want).abs().max() <= 2e-5 * max(1.0, want.abs().max().item()), (i, t - lo)
+            S = w[t][:, None, :] * S + kv
+        assert (left[i] - S).abs().max() <= 2e-5 * max(1.0, S.abs().max().item()), i
+
+
 @pytest.mark.parametrize("dtype", DTYPES)
 @pytest.mark.parametrize("taps", [1, 2, 3, 4, 5, 9])
 def test_the_convolution_reaches_back_over_steps_and_no_farther(dtype, taps):

@@ -22,13 +22,12 @@
 // COLS neighbouring columns, lane l the key channels 4l .. 4l + 3, 64 + 4l .. of each (runs of four, for
 // 16-byte accesses), so that a key, query or decay once loaded serves COLS columns.  One block per
 // (sequence, head, 16 columns) walks the sequence's tokens of the step in order.  The tokens come
-// through a ring of buffers in shared memory, filled by asynchronous 16-byte copies.  Eight
-// tokens are worked on together: their state updates follow one another, but their partial sums are
-// reduced over the lanes together, by halving: at every step a lane hands half of its sums to its partner
-// and keeps the other half, so that in the end each lane holds finished sums of its own tokens and columns
-// (15 or 30 shuffles for eight tokens where a butterfly per token takes 32 per column).  What is left of
-// a stage is reduced token by token in the same order of additions.  A row's result depends on
-// its sequence's own tokens only, in an order fixed by the sizes.
+// through a ring of buffers in shared memory, filled by asynchronous 16-byte copies: a warp copies whole
+// tokens, a lane the same pieces of each.  A token's sums over the lanes are not reduced one by one
+// (each would be a chain of shuffles that the next token waits behind): every lane leaves its share in
+// shared memory, and once a stage of tokens is through, each lane adds up the 16 shares of some
+// (token, column) pairs and writes their results.  A row's result depends on its sequence's own
+// tokens only, in an order fixed by the sizes.
 #include <math.h>
 
 #include "linear_attention.cuh"
@@ -37,10 +36,12 @@ namespace {
 
 constexpr int kLanes = kRecurrenceLanes;
 constexpr int kColumns = kRecurrenceColumns;  // columns of S per block
-constexpr int kGroup = 8;                     // tokens whose sums are reduced together
+constexpr int kGroup = 8;                     // tokens between whose loads no store stands
 // tokens per buffer, and buffers: fewer tokens for long keys, so that the ring fits
 constexpr int stage_tokens(int per) { return per <= 8 ? 16 : 8; }
 constexpr int kBuffers = 3;
+// floats between the shares of neighbouring columns: the two column groups of a warp store without bank conflicts
+constexpr int share_stride(int cols) { return cols == 2 ? 24 : 20; }
 
 __device__ __forceinline__ void copy16_async(void* smem, const void* gmem) {
     asm volatile("cp.async.cg.shared.global [%0], [%1], 16;\n" ::"r"((uint32_t)__cvta_generic_to_shared(smem)), "l"(gmem));
@@ -99,28 +100,6 @@ __global__ void linear_attention_prepare_kernel(float* __restrict__ prepared, co
     prepared[e] = v;
 }
 
-// N sums per lane, to be added over the 16 lanes of a group: the sum at index i ends on the lane
-// whose bits, high to low, are the high bits of i; a lane is left with N / 16 of them (one, if N < 16).
-template <int N>
-__device__ __forceinline__ void reduce_by_halving(float (&part)[N], int lane) {
-    int n = N;
-#pragma unroll
-    for (int off = kLanes / 2; off > 0; off >>= 1) {
-        if (n > 1) {
-            n >>= 1;
-            const bool upper = (lane & off) != 0;
-#pragma unroll
-            for (int i = 0; i < N / 2; ++i) {
-                if (i >= n) break;
-                const float give = upper ? part[i] : part[i + n], keep = upper ? part[i + n] : part[i];
-                part[i] = keep + __shfl_xor_sync(0xffffffffu, give, off);
-            }
-        } else {
-            part[0] += __shfl_xor_sync(0xffffffffu, part[0], off);
-        }
-    }
-}
-
 // PER: key channels per lane (a multiple of 4); KP = 16 * PER: the padded key size.  COLS: columns per lane.
 template <int PER, int COLS, int KIND>
 __global__ void __launch_bounds__(kLanes * kColumns / COLS) linear_attention_kernel(
@@ -135,9 +114,10 @@ __global__ void __launch_bounds__(kLanes * kColumns / COLS) linear_attention_ker
     constexpr int TAIL = KIND >= kBonusRead ? kRecurrenceTail : 0;
     constexpr int V_AT = PARTS * KP, TAIL_AT = V_AT + kColumns;
     constexpr int ROW = V_AT + kColumns + TAIL;         // floats of one staged token
-    constexpr int PIECES = ROW / 4;
-    constexpr int SUMS = kGroup * COLS, LEFT = SUMS > kLanes ? SUMS / kLanes : 1;
-    extern __shared__ __align__(16) float stage_mem[];  // [kBuffers][kStage][ROW]
+    constexpr int PIECES = ROW / 4, WARPS = kThreads / 32, PER_LANE = (PIECES + 31) / 32;
+    constexpr int SHARE = share_stride(COLS), WARP_COLS = 2 * COLS;
+    extern __shared__ __align__(16) float stage_mem[];  // [kBuffers][kStage][ROW], then the shares [kStage][kColumns][SHARE]
+    float* shares = stage_mem + (size_t)kBuffers * kStage * ROW;
     const int seq = blockIdx.z, head = blockIdx.y;
     const int col0 = blockIdx.x * kColumns;
     const int lane = threadIdx.x % kLanes, group = threadIdx.x / kLanes;
@@ -147,20 +127,33 @@ __global__ void __launch_bounds__(kLanes * kColumns / COLS) linear_attention_ker
     const int slot = slots[seq];
     float* S = state + ((size_t)slot * n_heads + head) * (size_t)value_dim * key_dim;
     const int unit = head / heads_per_unit, n_units = n_heads / heads_per_unit;
-    const float* key_src = keys + ((size_t)row0 * n_units + unit) * key_stride;
-    const float* value_src = values + ((size_t)row0 * n_heads + head) * value_stride;
     const size_t key_step = (size_t)n_units * key_stride, value_step = (size_t)n_heads * value_stride;
     const int n_tokens = row1 - row0;
+    const int warp = threadIdx.x >> 5, warp_lane = threadIdx.x & 31;
 
+    // a lane's pieces of a token: where each lies in its row, and how far apart rows are
+    const float* piece_src[PER_LANE];
+    size_t piece_step[PER_LANE];
+#pragma unroll
+    for (int j = 0; j < PER_LANE; ++j) {
+        const int c = (warp_lane + 32 * j) * 4;
+        if (c < V_AT) {
+            piece_src[j] = keys + ((size_t)row0 * n_units + unit) * key_stride + c;
+            piece_step[j] = key_step;
+        } else {
+            piece_src[j] = values + ((size_t)row0 * n_heads + head) * value_stride +
+                           (TAIL != 0 && c >= TAIL_AT ? vp + (c - TAIL_AT) : col0 + (c - V_AT));
+            piece_step[j] = value_step;
+        }
+    }
     auto issue = [&](int stage) {
         const int first = stage * kStage, n = min(kStage, n_tokens - first);
-        float* dst = stage_mem + (size_t)(stage % kBuffers) * kStage * ROW;
-        for (int piece = threadIdx.x; piece < n * PIECES; piece += kThreads) {
-            const int t = piece / PIECES, c = (piece - t * PIECES) * 4;
-            const float* src;
-            if (c < V_AT) src = key_src + (size_t)(first + t) * key_step + c;
-            else src = value_src + (size_t)(first + t) * value_step + (TAIL != 0 && c >= TAIL_AT ? vp + (c - TAIL_AT) : col0 + (c - V_AT));
-            copy16_async(dst + piece * 4, src);
+        float* dst = stage_mem + (size_t)(stage % kBuffers) * kStage * ROW + warp_lane * 4;
+        for (int t = warp; t < n; t += WARPS) {
+#pragma unroll
+            for (int j = 0; j < PER_LANE; ++j)
+                if (32 * (j + 1) <= PIECES || warp_lane + 32 * j < PIECES)
+                    copy16_async(dst + t * ROW + 128 * j, piece_src[j] + (size_t)(first + t) * piece_step[j]);
         }
     };
     const int n_stages = (n_tokens + kStage - 1) / kStage;
@@ -170,14 +163,21 @@ __global__ void __launch_bounds__(kLanes * kColumns / COLS) linear_attention_ker
         copy_commit();
     }
 
+    const bool whole = key_dim % 4 == 0 && ((uintptr_t)state & 15) == 0;
     float s[COLS][PER];
 #pragma unroll
     for (int c = 0; c < COLS; ++c) {
         const float* src = S + (size_t)min(own_col + c, value_dim - 1) * key_dim;     // idle columns mirror the last one and store nothing
 #pragma unroll
-        for (int i = 0; i < PER; ++i) {
-            const int d = (i / 4) * (4 * kLanes) + lane * 4 + (i & 3);
-            s[c][i] = d < key_dim ? src[d] : 0.f;
+        for (int i = 0; i < PER; i += 4) {
+            const int d = (i / 4) * (4 * kLanes) + lane * 4;
+            if (whole) {                      // a run of four is inside the key or outside as a whole
+                const float4 x = d < key_dim ? *reinterpret_cast<const float4*>(src + d) : make_float4(0.f, 0.f, 0.f, 0.f);
+                s[c][i] = x.x; s[c][i + 1] = x.y; s[c][i + 2] = x.z; s[c][i + 3] = x.w;
+            } else {
+#pragma unroll
+                for (int j = 0; j < 4; ++j) s[c][i + j] = d + j < key_dim ? src[d + j] : 0.f;
+            }
         }
     }
     const float own = per_head != nullptr ? per_head[head] : 0.f;      // the constant decay, or the skip's factor
@@ -208,23 +208,15 @@ __global__ void __launch_bounds__(kLanes * kColumns / COLS) linear_attention_ker
             for (int c = 0; c < COLS; ++c) {
                 float* x = s[c] + i;
                 if (KIND == kBonusRead) sums[c] += x[0] * q.x + x[1] * q.y + x[2] * q.z + x[3] * q.w;
-                x[0] = a.x * x[0] + k.x * v[c];
-                x[1] = a.y * x[1] + k.y * v[c];
-                x[2] = a.z * x[2] + k.z * v[c];
-                x[3] = a.w * x[3] + k.w * v[c];
+                x[0] = fmaf(a.x, x[0], k.x * v[c]);      // (one multiply-add links a token's state to the next)
+                x[1] = fmaf(a.y, x[1], k.y * v[c]);
+                x[2] = fmaf(a.z, x[2], k.z * v[c]);
+                x[3] = fmaf(a.w, x[3], k.w * v[c]);
                 if (KIND != kBonusRead) sums[c] += x[0] * q.x + x[1] * q.y + x[2] * q.z + x[3] * q.w;
             }
         }
     };
-    // the finished sum of column c of this lane's group, for the stage's token at tok, row `row`
-    auto store = [&](const float* tok, int row, int c, float sum) {
-        const int column = own_col + c;
-        if (column >= value_dim) return;
-        float y = sum * q_scale;
-        if (KIND == kBonusRead) y += tok[TAIL_AT] * tok[V_AT + group * COLS + c];
-        if (KIND == kSteppedDecay) y += own * tok[V_AT + group * COLS + c];
-        o[((size_t)row * n_heads + head) * value_dim + column] = y;
-    };
+    float* own_share = shares + (size_t)group * COLS * SHARE + lane;
 
     for (int stage = 0; stage < n_stages; ++stage) {
         copy_wait<kBuffers - 2>();
@@ -236,35 +228,38 @@ __global__ void __launch_bounds__(kLanes * kColumns / COLS) linear_attention_ker
         int t0 = 0;
 #pragma unroll 1
         for (; t0 + kGroup <= n; t0 += kGroup) {
-            float part[SUMS];
+            float part[kGroup][COLS];
 #pragma unroll
-            for (int t = 0; t < kGroup; ++t) {
-                float sums[COLS];
-                advance(src + (t0 + t) * ROW, sums);
+            for (int t = 0; t < kGroup; ++t) advance(src + (t0 + t) * ROW, part[t]);
 #pragma unroll
-                for (int c = 0; c < COLS; ++c) part[t * COLS + c] = sums[c];
-            }
-            reduce_by_halving<SUMS>(part, lane);
-            const int index = SUMS >= kLanes ? lane * LEFT : lane / (kLanes / SUMS);
-            if (SUMS >= kLanes || lane % (kLanes / (SUMS < kLanes ? SUMS : 1)) == 0) {
+            for (int t = 0; t < kGroup; ++t)
 #pragma unroll
-                for (int j = 0; j < LEFT; ++j) {
-                    const int t = t0 + (index + j) / COLS;
-                    store(src + t * ROW, row0 + first + t, (index + j) % COLS, part[j]);
-                }
-            }
+                for (int c = 0; c < COLS; ++c) own_share[(size_t)((t0 + t) * kColumns + c) * SHARE] = part[t][c];
         }
 #pragma unroll 1
         for (; t0 < n; ++t0) {
-            float sums[COLS];
-            advance(src + t0 * ROW, sums);
+            float part[COLS];
+            advance(src + t0 * ROW, part);
 #pragma unroll
-            for (int off = kLanes / 2; off > 0; off >>= 1)
+            for (int c = 0; c < COLS; ++c) own_share[(size_t)(t0 * kColumns + c) * SHARE] = part[c];
+        }
+        __syncwarp();
+        // the stage's read-outs: this warp's columns, a (token, column) pair per lane and turn
+        for (int i = warp_lane; i < n * WARP_COLS; i += 32) {
+            const int t = i / WARP_COLS, c = warp * WARP_COLS + i % WARP_COLS;
+            const float* share = shares + (size_t)(t * kColumns + c) * SHARE;
+            float sum = 0.f;
 #pragma unroll
-                for (int c = 0; c < COLS; ++c) sums[c] += __shfl_xor_sync(0xffffffffu, sums[c], off);
-            if (lane == 0) {
-#pragma unroll
-                for (int c = 0; c < COLS; ++c) store(src + t0 * ROW, row0 + first + t0, c, sums[c]);
+            for (int l = 0; l < kLanes; l += 4) {
+                const float4 x = *reinterpret_cast<const float4*>(share + l);
+                sum += (x.x + x.y) + (x.z + x.w);
+            }
+            if (col0 + c < value_dim) {
+                const float* tok = src + t * ROW;
+                float y = sum * q_scale;
+                if (KIND == kBonusRead) y += tok[TAIL_AT] * tok[V_AT + c];
+                if (KIND == kSteppedDecay) y += own * tok[V_AT + c];
+                o[((size_t)(row0 + first + t) * n_heads + head) * value_dim + col0 + c] = y;
             }
         }
     }
@@ -273,9 +268,15 @@ __global__ void __launch_bounds__(kLanes * kColumns / COLS) linear_attention_ker
         if (own_col + c >= value_dim) break;
         float* dst = S + (size_t)(own_col + c) * key_dim;
 #pragma unroll
-        for (int i = 0; i < PER; ++i) {
-            const int d = (i / 4) * (4 * kLanes) + lane * 4 + (i & 3);
-            if (d < key_dim) dst[d] = s[c][i];
+        for (int i = 0; i < PER; i += 4) {
+            const int d = (i / 4) * (4 * kLanes) + lane * 4;
+            if (whole) {
+                if (d < key_dim) *reinterpret_cast<float4*>(dst + d) = make_float4(s[c][i], s[c][i + 1], s[c][i + 2], s[c][i + 3]);
+            } else {
+#pragma unroll
+                for (int j = 0; j < 4; ++j)
+                    if (d + j < key_dim) dst[d + j] = s[c][i + j];
+            }
         }
     }
 }
@@ -284,7 +285,7 @@ template <int PER, int COLS, int KIND>
 void launch_one(const RecurrenceArgs& a, cudaStream_t stream) {
     constexpr int KP = kLanes * PER, kStage = stage_tokens(PER);
     constexpr int ROW = (KIND == kChannelDecay || KIND == kBonusRead ? 3 : 2) * KP + kColumns + (KIND >= kBonusRead ? kRecurrenceTail : 0);
-    const size_t smem = kBuffers * (size_t)kStage * ROW * sizeof(float);
+    const size_t smem = (size_t)kStage * (kBuffers * ROW + kColumns * share_stride(COLS)) * sizeof(float);
     const dim3 grid((a.value_dim + kColumns - 1) / kColumns, a.n_heads, a.n_seqs);
     auto kernel = linear_attention_kernel<PER, COLS, KIND>;
     if (smem > 48 * 1024) cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
@@ -304,9 +305,14 @@ void launch_columns(const RecurrenceArgs& a, int columns, cudaStream_t stream) {
 
 template <int KIND>
 void launch_kind(const RecurrenceArgs& a, cudaStream_t stream) {
+    // Four columns a lane load less per multiply-add, two leave twice as many warps: with fewer than 256
+    // blocks the latter win (one prompt of 2,048 tokens, 32 heads of 64: 208 against 263 us; four of them 618
+    // against 607; 64 heads of 64 over a state of 128: 366 against 364 us, four prompts 1,322 against 1,171).
+    const long long blocks = (long long)(padded_values(a.value_dim) / kColumns) * a.n_heads * a.n_seqs;
+    const int columns = g_columns ? g_columns : blocks >= 256 ? 4 : 2;
     switch (recurrence_per_lane(a.key_dim)) {
-        case 4: return launch_columns<4, KIND>(a, g_columns ? g_columns : 2, stream);
-        case 8: return launch_columns<8, KIND>(a, g_columns ? g_columns : 2, stream);
+        case 4: return launch_columns<4, KIND>(a, columns, stream);
+        case 8: return launch_columns<8, KIND>(a, columns, stream);
         case 16: return launch_one<16, 2, KIND>(a, stream);
         default: return launch_one<32, 1, KIND>(a, stream);
     }

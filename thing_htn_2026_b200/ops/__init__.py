@@ -732,11 +732,14 @@ SKINNY_ANY_ROWS_COLUMNS = 16
 
 
 def linear(x: torch.Tensor, weight: torch.Tensor, out_dtype: Optional[torch.dtype] = None,
-           err: Optional[torch.Tensor] = None, bias: Optional[torch.Tensor] = None) -> torch.Tensor:
+           err: Optional[torch.Tensor] = None, bias: Optional[torch.Tensor] = None,
+           rows_alone: bool = True) -> torch.Tensor:
     """x [M, K] @ weight[N, K]^T.  float32: this library's FFMA kernel.  bfloat16 with few
     rows and a deep reduction or a tall weight: this library's weight-streaming kernel
     (``err``: the step's device error word for its bounded waits).  bfloat16 with a float32 result
-    of at most 64 columns (a router, a gate; with many rows of at most 16): this library's warp-per-row kernel.  bfloat16 otherwise: the
+    of at most 64 columns (a router, a gate): this library's warp-per-row kernel, in which a row's result does not
+    depend on the rows beside it by a bit (``rows_alone`` False: rounding may, and many rows of more than
+    a few columns go to the vendor library).  bfloat16 otherwise: the
     vendor library's tensor-core product with float32 accumulation (the reference's choice,
     engine/engine.py:341-350).  ``out_dtype=torch.float32`` keeps the accumulator's
     precision (used for logits).  ``bias`` (of the activation type, ``[N]``) is added to every row:
@@ -768,7 +771,7 @@ def linear(x: torch.Tensor, weight: torch.Tensor, out_dtype: Optional[torch.dtyp
     if x.dtype != torch.bfloat16:
         raise KernelError(f"linear: dtype {x.dtype} is not supported")
     if (out_dtype == torch.float32 and lib().thn_linear_skinny_supported(weight.shape[0], x.shape[1])
-            and (x.shape[0] < SKINNY_MAX_ROWS or weight.shape[0] <= SKINNY_ANY_ROWS_COLUMNS)
+            and (rows_alone or x.shape[0] < SKINNY_MAX_ROWS or weight.shape[0] <= SKINNY_ANY_ROWS_COLUMNS)
             and (x.data_ptr() | weight.data_ptr()) % 16 == 0):
         # a router or a gate: a few float32 outputs per row, on this library's warp-per-row kernel
         out = torch.empty((x.shape[0], weight.shape[0]), dtype=torch.float32, device=x.device)

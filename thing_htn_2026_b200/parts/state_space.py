@@ -77,7 +77,7 @@ class StateSpaceMixer:
     def forward(self, x: torch.Tensor, ctx: StepContext, entry: ScheduleEntry) -> torch.Tensor:
         state, ring = ctx.cache.state_view(entry.cache, 0), ctx.cache.state_view(entry.cache, 1)
         proj = ops.linear(x, self.w_in, err=ctx.err)
-        dt = ops.linear(x, self.w_dt, out_dtype=torch.float32, err=ctx.err)
+        dt = ops.linear(x, self.w_dt, out_dtype=torch.float32, err=ctx.err, rows_alone=False)
         y = ops.state_space(proj, self.inner, dt, self.shape, state, ring, ctx.rows, ctx.cache.seq_lens)
         n = ops.gated_group_norm(y, proj, 0, self.gain, self.eps, self.parts, self.dtype)
         return ops.linear(n, self.w_o, err=ctx.err)

@@ -74,7 +74,7 @@ class TimeMixing:
         state, shift = ctx.cache.state_view(entry.cache, 0), ctx.cache.state_view(entry.cache, 1)
         blends = ops.token_shift(x, self.mu, shift, ctx.rows, ctx.cache.seq_lens)
         planes = ops.linear_batched(blends[:len(WIDE)], self.w_wide)
-        low = ops.linear(blends[len(WIDE)], self.w1, out_dtype=torch.float32, err=ctx.err)
+        low = ops.linear(blends[len(WIDE)], self.w1, out_dtype=torch.float32, err=ctx.err, rows_alone=False)
         if ctx.rows.max_q_len == 1:
             y = ops.wkv_decode(planes, low, self.w2, self.w0, self.u, self.gain, self.eps, state, ctx.rows, self.n_heads, self.dim)
         else:
