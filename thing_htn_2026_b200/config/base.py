@@ -90,12 +90,14 @@ class ScheduleEntry:
     its weights are then shared).  ``cache`` is the id of the cache entry the
     mixer works on; two schedule entries with the same ``cache`` share it, and
     only the entry with ``writes_cache`` appends to it (the other one reads what
-    the first wrote).
+    the first wrote).  ``adds_start``: the stream as the embedding started it is
+    added to the stream ahead of this execution (a later pass over looped layers).
     """
 
     layer: int
     cache: int
     writes_cache: bool = True
+    adds_start: bool = False
 
 
 @dataclass(frozen=True)
@@ -132,6 +134,17 @@ class ModelPlan:
     @property
     def n_cache_entries(self) -> int:
         return 1 + max((e.cache for e in self.schedule), default=-1)
+
+
+def looped_schedule(n_layers: int, start: int = 0, stop: int = 0, times: int = 1) -> Tuple[ScheduleEntry, ...]:
+    """The layers in order, ``start`` to ``stop - 1`` run ``times`` times in a row with the same weights.
+    Every execution has a cache entry of its own; every pass but the first adds the stream's start ahead of
+    its first layer."""
+    runs = [(i, False) for i in range(start)]
+    for go in range(times):
+        runs += [(i, go > 0 and i == start) for i in range(start, stop)]
+    runs += [(i, False) for i in range(max(start, stop), n_layers)]
+    return tuple(ScheduleEntry(layer=layer, cache=cache, adds_start=again) for cache, (layer, again) in enumerate(runs))
 
 
 class ModelConfig:

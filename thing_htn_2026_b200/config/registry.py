@@ -68,12 +68,14 @@ def _register_builtin() -> None:
     from .futepel import FutepelConfig
     from .lanilix import LanilixConfig
     from .qwen3 import Qwen3Config
+    from .turutar import TurutarConfig
     register_architecture(Qwen3Config.architecture, Qwen3Config, _decoder_model)
     register_architecture(LanilixConfig.architecture, LanilixConfig, _decoder_model)
     register_architecture(BunudraConfig.architecture, BunudraConfig, _decoder_model)
     register_architecture(DitilixConfig.architecture, DitilixConfig, _decoder_model)
     register_architecture(DubazenConfig.architecture, DubazenConfig, _decoder_model)
     register_architecture(FutepelConfig.architecture, FutepelConfig, _decoder_model)
+    register_architecture(TurutarConfig.architecture, TurutarConfig, _decoder_model)
 
 
 _register_builtin()

@@ -4,7 +4,8 @@
 // key part of `rot` entries that is to be rotated by the token's position.
 //
 //   latent_norm      c = latent / sqrt(mean(latent^2) + eps) * w   -> [rows, rank], the operand of
-//                    the up-projection that gives every head's unrotated key and its value.
+//                    the up-projection that gives every head's unrotated key and its value.  Where
+//                    the queries are read out of a latent of their own, both are normalised in one launch.
 //   latent_assemble  from the row's queries [heads][plain | rot], the up-projection's result
 //                    [heads * plain keys | heads * values] and the shared key part: queries with
 //                    their last `rot` entries rotated; per head the key [plain | rotated shared
@@ -19,22 +20,30 @@
 
 namespace {
 
+// One latent of a projected row: where it starts in the row, its size, its gain and its output.
+struct Latent {
+    void* out;
+    const float* gain;
+    long long offset;
+    int rank;
+};
+
 template <typename T>
-__global__ void __launch_bounds__(128) latent_norm_kernel(T* __restrict__ out, const T* __restrict__ src,
-                                                          long long src_stride, const float* __restrict__ gain, float eps,
-                                                          int rank) {
+__global__ void __launch_bounds__(128) latent_norm_kernel(Latent one, Latent two, const T* __restrict__ src,
+                                                          long long src_stride, float eps) {
     pdl_launch_dependents();
     pdl_wait();
     __shared__ float scratch[33];
-    const T* row = src + (size_t)blockIdx.x * src_stride;
+    const Latent l = blockIdx.y ? two : one;
+    const T* row = src + (size_t)blockIdx.x * src_stride + l.offset;
+    T* out = (T*)l.out + (size_t)blockIdx.x * l.rank;
     float ss = 0.f;
-    for (int i = threadIdx.x; i < rank; i += blockDim.x) {
+    for (int i = threadIdx.x; i < l.rank; i += blockDim.x) {
         const float v = to_f32<T>(row[i]);
         ss += v * v;
     }
-    const float r = 1.0f / sqrtf(block_sum(ss, scratch) / (float)rank + eps);
-    for (int i = threadIdx.x; i < rank; i += blockDim.x)
-        out[(size_t)blockIdx.x * rank + i] = from_f32<T>(to_f32<T>(row[i]) * r * gain[i]);
+    const float r = 1.0f / sqrtf(block_sum(ss, scratch) / (float)l.rank + eps);
+    for (int i = threadIdx.x; i < l.rank; i += blockDim.x) out[i] = from_f32<T>(to_f32<T>(row[i]) * r * l.gain[i]);
 }
 
 template <typename T>
@@ -193,17 +202,22 @@ __global__ void __launch_bounds__(256) latent_assemble_vec_kernel(
 
 }  // namespace
 
-// src: rows of the activation type, `rank` entries each, src_stride elements apart; gain float32
-// [rank]; out [rows, rank] of the activation type.
-THN_API int thn_latent_norm(void* out, const void* src, long long src_stride, const float* gain, float eps, int rows,
-                            int rank, int dtype, cudaStream_t stream) {
-    THN_CHECK_ARG(rows >= 0 && rank > 0 && src_stride >= rank && eps > 0.f && gain, "latent_norm: bad arguments");
+// src: rows of the activation type, src_stride elements apart, with a latent of `rank` entries from column
+// `offset` and, if out2 is given, another one of rank2 from offset2; gains float32 [rank]; out [rows, rank] of
+// the activation type.
+THN_API int thn_latent_norm(void* out, long long offset, const float* gain, int rank, void* out2, long long offset2,
+                            const float* gain2, int rank2, const void* src, long long src_stride, float eps, int rows, int dtype,
+                            cudaStream_t stream) {
+    THN_CHECK_ARG(rows >= 0 && rank > 0 && offset >= 0 && src_stride >= offset + rank && eps > 0.f && gain, "latent_norm: bad arguments");
+    THN_CHECK_ARG(out2 == nullptr || (rank2 > 0 && offset2 >= 0 && src_stride >= offset2 + rank2 && gain2),
+                  "latent_norm: bad arguments of the second latent");
     if (rows == 0) return THN_OK;
+    const Latent one{out, gain, offset, rank}, two{out2, gain2, offset2, rank2};
+    const dim3 grid(rows, out2 ? 2 : 1);
     if (dtype == THN_F32)
-        thn_launch(latent_norm_kernel<float>, rows, 128, 0, stream, (float*)out, (const float*)src, src_stride, gain, eps, rank);
+        thn_launch(latent_norm_kernel<float>, grid, 128, 0, stream, one, two, (const float*)src, src_stride, eps);
     else if (dtype == THN_BF16)
-        thn_launch(latent_norm_kernel<__nv_bfloat16>, rows, 128, 0, stream, (__nv_bfloat16*)out, (const __nv_bfloat16*)src,
-                   src_stride, gain, eps, rank);
+        thn_launch(latent_norm_kernel<__nv_bfloat16>, grid, 128, 0, stream, one, two, (const __nv_bfloat16*)src, src_stride, eps);
     else
         THN_CHECK_ARG(false, "latent_norm: unknown dtype %d", dtype);
     return thn_launch_status("latent_norm");

@@ -1,7 +1,10 @@
 // Norms around a residual stream that is kept in float32 whatever the activation type is,
 // with an optional norm of the branch output before it is added:
 //
-//     h <- h + m B(d + d2)   (d2, a second branch output, may be absent; m is 1 unless given)
+//     h <- h + (s p + s' p') + m B(d + d2) + a
+//                      (each of these may be absent: p and p', branch outputs that are added first, entry by
+//                      entry times s and s' (layer scale); d2, a second output of the branch; a, rows of
+//                      float32 that are added as they are; m is 1 unless given)
 //                      B(d) = d                                                  (post kind 0)
 //                      B(d) = d / sqrt(mean(d^2) + eps_b) * (o_b + w_b)          (post kind 1, RMS)
 //                      B(d) = (d - mean d) / sqrt(var d + eps_b) * (o_b + w_b) + b_b   (post kind 2, layer norm)
@@ -32,6 +35,15 @@ struct NormArgs {
     float eps;
     int kind;     // 0 none, 1 RMS, 2 layer norm, 3 (output only) the stream as it is
     int groups;   // kind 1 as an output: equal consecutive parts with statistics of their own (1: the whole row)
+};
+
+// What is added to the stream besides the branch d; all of it may be absent (null).
+struct AddArgs {
+    const void* d2;              // a second output of the branch, of the activation type
+    float mult;                  // the factor on the branch
+    const void *first, *second;  // outputs that are added ahead of the branch, of the activation type
+    const float *scale1, *scale2;  // [width]: the factors on their entries
+    const float* rows;           // float32 [rows, width]
 };
 
 // 1 / sqrt(mean(part^2) + eps) of each of `groups` equal parts of the staged row, into rstd[];
@@ -66,13 +78,24 @@ __device__ __forceinline__ float2 row_statistics(const float* row, int width, in
 
 template <typename T>
 __global__ void __launch_bounds__(kThreads) residual_norm_kernel(
-    T* __restrict__ y, float* __restrict__ h, const T* __restrict__ d, const T* __restrict__ d2, float mult,
-    NormArgs post, NormArgs out, int width, int h_is_new) {
+    T* __restrict__ y, float* __restrict__ h, const T* __restrict__ d, AddArgs add, NormArgs post, NormArgs out, int width,
+    int h_is_new) {
     pdl_launch_dependents();
     pdl_wait();
     extern __shared__ float row[];
     __shared__ float scratch[33];
     const size_t base = (size_t)blockIdx.x * width;
+    const T *d2 = (const T*)add.d2, *p1 = (const T*)add.first, *p2 = (const T*)add.second;
+    // the stream with what is added ahead of the branch
+    auto stream = [&](int i) {
+        float v = h_is_new ? 0.f : h[base + i];
+        if (p1) {
+            float s = to_f32<T>(p1[base + i]) * add.scale1[i];
+            if (p2) s = fmaf(to_f32<T>(p2[base + i]), add.scale2[i], s);
+            v = __fadd_rn(v, s);
+        }
+        return v;
+    };
     if (d) {
         for (int i = threadIdx.x; i < width; i += kThreads)
             row[i] = d2 ? to_f32<T>(d[base + i]) + to_f32<T>(d2[base + i]) : to_f32<T>(d[base + i]);
@@ -87,13 +110,20 @@ __global__ void __launch_bounds__(kThreads) residual_norm_kernel(
                 v = (v - st.x) * st.y * (post.offset + post.gain[i]);
                 if (post.bias) v += post.bias[i];
             }
-            v *= mult;
-            if (!h_is_new) v = h[base + i] + v;
+            v *= add.mult;
+            if (!h_is_new || p1) v = stream(i) + v;
+            if (add.rows) v = __fadd_rn(v, add.rows[base + i]);
             h[base + i] = v;
             row[i] = v;
         }
     } else {
-        for (int i = threadIdx.x; i < width; i += kThreads) row[i] = h[base + i];
+        const bool changes = p1 || add.rows;
+        for (int i = threadIdx.x; i < width; i += kThreads) {
+            float v = stream(i);
+            if (add.rows) v = __fadd_rn(v, add.rows[base + i]);
+            if (changes) h[base + i] = v;
+            row[i] = v;
+        }
     }
     if (!out.kind) return;
     if (out.kind == 3) {
@@ -150,14 +180,45 @@ __device__ __forceinline__ void store8(__nv_bfloat16* p, const float (&v)[8]) {
 }
 
 __global__ void __launch_bounds__(kThreads) residual_norm_bf16x8_kernel(
-    __nv_bfloat16* __restrict__ y, float* __restrict__ h, const __nv_bfloat16* __restrict__ d,
-    const __nv_bfloat16* __restrict__ d2, float mult, NormArgs post, NormArgs out, int width, int h_is_new) {
+    __nv_bfloat16* __restrict__ y, float* __restrict__ h, const __nv_bfloat16* __restrict__ d, AddArgs add, NormArgs post,
+    NormArgs out, int width, int h_is_new) {
     pdl_launch_dependents();
     pdl_wait();
     extern __shared__ __align__(16) float row[];
     __shared__ float scratch[33];
     const size_t base = (size_t)blockIdx.x * width;
     float v[8], u[8];
+    const __nv_bfloat16 *d2 = (const __nv_bfloat16*)add.d2, *p1 = (const __nv_bfloat16*)add.first,
+                        *p2 = (const __nv_bfloat16*)add.second;
+    // eight entries of the stream with what is added ahead of the branch
+    auto stream = [&](int i, float (&x)[8]) {
+        if (h_is_new) {
+#pragma unroll
+            for (int e = 0; e < 8; ++e) x[e] = 0.f;
+        } else {
+            load8(h + base + i, x);
+        }
+        if (!p1) return;
+        float s[8], w[8], f[8];
+        load8(p1 + base + i, s);
+        load8(add.scale1 + i, f);
+#pragma unroll
+        for (int e = 0; e < 8; ++e) s[e] *= f[e];
+        if (p2) {
+            load8(p2 + base + i, w);
+            load8(add.scale2 + i, f);
+#pragma unroll
+            for (int e = 0; e < 8; ++e) s[e] = fmaf(w[e], f[e], s[e]);
+        }
+#pragma unroll
+        for (int e = 0; e < 8; ++e) x[e] = __fadd_rn(x[e], s[e]);
+    };
+    auto add_rows = [&](int i) {
+        if (!add.rows) return;
+        load8(add.rows + base + i, u);
+#pragma unroll
+        for (int e = 0; e < 8; ++e) v[e] = __fadd_rn(v[e], u[e]);
+    };
     if (d) {
         if (post.kind) {
             for (int i = threadIdx.x * 8; i < width; i += kThreads * 8) {
@@ -193,18 +254,22 @@ __global__ void __launch_bounds__(kThreads) residual_norm_bf16x8_kernel(
                 }
             }
 #pragma unroll
-            for (int e = 0; e < 8; ++e) v[e] *= mult;
-            if (!h_is_new) {
-                load8(h + base + i, u);
+            for (int e = 0; e < 8; ++e) v[e] *= add.mult;
+            if (!h_is_new || p1) {
+                stream(i, u);
 #pragma unroll
                 for (int e = 0; e < 8; ++e) v[e] = u[e] + v[e];
             }
+            add_rows(i);
             store8(h + base + i, v);
             store8(row + i, v);
         }
     } else {
+        const bool changes = p1 || add.rows;
         for (int i = threadIdx.x * 8; i < width; i += kThreads * 8) {
-            load8(h + base + i, v);
+            stream(i, v);
+            add_rows(i);
+            if (changes) store8(h + base + i, v);
             store8(row + i, v);
         }
     }
@@ -241,21 +306,22 @@ __global__ void __launch_bounds__(kThreads) residual_norm_bf16x8_kernel(
 inline bool aligned16(const void* p) { return ((uintptr_t)p & 15) == 0; }
 
 template <typename T>
-int launch(void* y, float* h, const void* d, const void* d2, float mult, NormArgs post, NormArgs out, int rows, int width,
-           int h_is_new, cudaStream_t stream) {
+int launch(void* y, float* h, const void* d, AddArgs add, NormArgs post, NormArgs out, int rows, int width, int h_is_new,
+           cudaStream_t stream) {
     const size_t smem = (size_t)(width + (out.groups > 1 ? out.groups : 0)) * sizeof(float);
     THN_UNSUPPORTED_IF(smem > 200 * 1024, "residual_norm: rows of %d values do not fit shared memory", width);
     if (std::is_same<T, __nv_bfloat16>::value && width % 8 == 0 && aligned16(y) && aligned16(h) && aligned16(d) &&
-        aligned16(d2) && aligned16(post.gain) && aligned16(post.bias) && aligned16(out.gain) && aligned16(out.bias)) {
+        aligned16(add.d2) && aligned16(add.first) && aligned16(add.second) && aligned16(add.scale1) && aligned16(add.scale2) &&
+        aligned16(add.rows) && aligned16(post.gain) && aligned16(post.bias) && aligned16(out.gain) && aligned16(out.bias)) {
         if (smem > 32 * 1024)
             cudaFuncSetAttribute(residual_norm_bf16x8_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
         thn_launch(residual_norm_bf16x8_kernel, rows, kThreads, smem, stream, (__nv_bfloat16*)y, h, (const __nv_bfloat16*)d,
-                   (const __nv_bfloat16*)d2, mult, post, out, width, h_is_new);
+                   add, post, out, width, h_is_new);
         return thn_launch_status("residual_norm");
     }
     if (smem > 32 * 1024)
         cudaFuncSetAttribute(residual_norm_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-    thn_launch(residual_norm_kernel<T>, rows, kThreads, smem, stream, (T*)y, h, (const T*)d, (const T*)d2, mult, post, out, width, h_is_new);
+    thn_launch(residual_norm_kernel<T>, rows, kThreads, smem, stream, (T*)y, h, (const T*)d, add, post, out, width, h_is_new);
     return thn_launch_status("residual_norm");
 }
 
@@ -375,23 +441,30 @@ __global__ void gated_head_norm_bf16_vec_kernel(__nv_bfloat16* __restrict__ out,
 }
 }  // namespace
 
-// h float32 [rows, width], updated in place when d is given (h_is_new: h is not read, it
-// becomes B(d)); d and y of the activation type; gains and biases float32 [width] (a bias may
-// be null).  post_kind 0: d is added as it is; kind 0: no y is written; kind 3: y is h rounded.
-// d2 (may be null): a second branch output, added to d before anything else; mult: the factor on
-// what is added to h; groups (kind 1 only, a divisor of width): parts of the row with statistics
-// of their own.
-THN_API int thn_residual_norm(void* y, float* h, const void* d, const void* d2, float mult, const float* post_gain,
-                              const float* post_bias, float post_offset, float post_eps, int post_kind, const float* gain,
-                              const float* bias, float offset, float eps, int kind, int groups, int rows, int width,
-                              int h_is_new, int dtype, cudaStream_t stream) {
+// h float32 [rows, width], updated in place when something is added (h_is_new: h is not read, it
+// becomes what is added); d, the outputs beside it and y of the activation type; gains and biases float32
+// [width] (a bias may be null).  post_kind 0: d is added as it is; kind 0: no y is written; kind 3: y is
+// h rounded.  d2 (may be null): a second output of the branch, added to d before anything else; mult: the
+// factor on the branch; first and second with scale1 and scale2 (float32 [width]; second or both may be
+// null): scale1 first + scale2 second is added to h ahead of the branch; add_rows (float32 [rows, width],
+// may be null): added to h behind it; groups (kind 1 only, a divisor of width): parts of the row with
+// statistics of their own.
+THN_API int thn_residual_norm(void* y, float* h, const void* d, const void* d2, float mult, const void* first,
+                              const float* scale1, const void* second, const float* scale2, const float* add_rows,
+                              const float* post_gain, const float* post_bias, float post_offset, float post_eps,
+                              int post_kind, const float* gain, const float* bias, float offset, float eps, int kind,
+                              int groups, int rows, int width, int h_is_new, int dtype, cudaStream_t stream) {
     THN_CHECK_ARG(rows >= 0 && width > 0, "residual_norm: bad sizes rows=%d width=%d", rows, width);
     THN_CHECK_ARG(d2 == nullptr || d != nullptr, "residual_norm: a second branch without a first");
+    THN_CHECK_ARG((first == nullptr) == (scale1 == nullptr) && (second == nullptr) == (scale2 == nullptr) &&
+                      (second == nullptr || first != nullptr),
+                  "residual_norm: scaled outputs come with their factors, the second with a first");
     THN_CHECK_ARG(groups >= 1 && width % groups == 0 && (groups == 1 || kind == 1),
                   "residual_norm: %d groups over rows of %d (an RMS norm of the stream only)", groups, width);
     THN_CHECK_ARG(post_kind >= 0 && post_kind <= 2 && kind >= 0 && kind <= 3, "residual_norm: norm kinds %d, %d", post_kind,
                   kind);
-    THN_CHECK_ARG(h != nullptr && (d != nullptr || kind != 0), "residual_norm: nothing to do");
+    THN_CHECK_ARG(h != nullptr && (d != nullptr || first != nullptr || add_rows != nullptr || kind != 0),
+                  "residual_norm: nothing to do");
     THN_CHECK_ARG(d != nullptr || !h_is_new, "residual_norm: a new residual stream needs a branch to start from");
     THN_CHECK_ARG(kind == 0 || y != nullptr, "residual_norm: an output norm without y");
     THN_CHECK_ARG(!(kind == 1 || kind == 2) || (gain != nullptr && eps > 0.f), "residual_norm: gain missing, or eps <= 0");
@@ -399,10 +472,86 @@ THN_API int thn_residual_norm(void* y, float* h, const void* d, const void* d2, 
     if (rows == 0) return THN_OK;
     const NormArgs post{post_gain, post_bias, post_offset, post_eps, d ? post_kind : 0, 1};
     const NormArgs out{gain, bias, offset, eps, kind, groups};
-    if (dtype == THN_F32) return launch<float>(y, h, d, d2, mult, post, out, rows, width, h_is_new, stream);
-    if (dtype == THN_BF16) return launch<__nv_bfloat16>(y, h, d, d2, mult, post, out, rows, width, h_is_new, stream);
+    const AddArgs add{d2, mult, first, second, scale1, scale2, add_rows};
+    if (dtype == THN_F32) return launch<float>(y, h, d, add, post, out, rows, width, h_is_new, stream);
+    if (dtype == THN_BF16) return launch<__nv_bfloat16>(y, h, d, add, post, out, rows, width, h_is_new, stream);
     THN_CHECK_ARG(false, "residual_norm: unknown dtype %d", dtype);
     return THN_OK;
+}
+
+// out[m] = table[token] / sqrt(mean(table[token]^2) + eps) * (offset + gain) in float32: token
+// embeddings that pass a norm as they start a residual stream kept in float32.  copy (may be null): a second
+// place for the same rows, for a model that adds the start of the stream again later.
+namespace {
+template <typename T>
+__global__ void __launch_bounds__(kThreads) embed_norm_kernel(float* __restrict__ out, float* __restrict__ copy,
+                                                              const T* __restrict__ table, const int* __restrict__ tokens,
+                                                              const float* __restrict__ gain, float offset, float eps,
+                                                              int width, int n_table_rows, int* __restrict__ err) {
+    pdl_launch_dependents();
+    pdl_wait();
+    extern __shared__ __align__(16) float row[];
+    __shared__ float scratch[33];
+    const int m = blockIdx.x;
+    int token = tokens[m];
+    if (token < 0 || token >= n_table_rows) {
+        if (threadIdx.x == 0 && err) atomicOr(err, THN_ERR_TOKEN_RANGE);
+        token = 0;
+    }
+    const T* src = table + (size_t)token * width;
+    const size_t base = (size_t)m * width;
+    const bool vec = width % 8 == 0 && (((uintptr_t)src | (uintptr_t)gain | (uintptr_t)out | (uintptr_t)copy) & 15) == 0;
+    float v[8], u[8];
+    if (vec) {
+        for (int i = threadIdx.x * 8; i < width; i += kThreads * 8) {
+            load8(src + i, v);
+            store8(row + i, v);
+        }
+    } else {
+        for (int i = threadIdx.x; i < width; i += kThreads) row[i] = to_f32<T>(src[i]);
+    }
+    __syncthreads();
+    const float r = row_statistics(row, width, 1, eps, scratch).y;
+    if (vec) {
+        for (int i = threadIdx.x * 8; i < width; i += kThreads * 8) {
+            load8(row + i, v);
+            load8(gain + i, u);
+#pragma unroll
+            for (int e = 0; e < 8; ++e) v[e] = v[e] * r * (offset + u[e]);
+            store8(out + base + i, v);
+            if (copy) store8(copy + base + i, v);
+        }
+    } else {
+        for (int i = threadIdx.x; i < width; i += kThreads) {
+            const float x = row[i] * r * (offset + gain[i]);
+            out[base + i] = x;
+            if (copy) copy[base + i] = x;
+        }
+    }
+}
+}  // namespace
+
+THN_API int thn_embed_norm(float* out, float* copy, const void* table, const int* tokens, const float* gain, float offset,
+                           float eps, int rows, int width, int n_table_rows, int dtype, int* err, cudaStream_t stream) {
+    THN_CHECK_ARG(rows >= 0 && width > 0 && n_table_rows > 0 && eps > 0.f && gain, "embed_norm: bad arguments rows=%d width=%d table=%d",
+                  rows, width, n_table_rows);
+    if (rows == 0) return THN_OK;
+    const size_t smem = (size_t)width * sizeof(float);
+    THN_UNSUPPORTED_IF(smem > 200 * 1024, "embed_norm: rows of %d values do not fit shared memory", width);
+    if (dtype == THN_F32) {
+        if (smem > 32 * 1024)
+            cudaFuncSetAttribute(embed_norm_kernel<float>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+        thn_launch(embed_norm_kernel<float>, rows, kThreads, smem, stream, out, copy, (const float*)table, tokens, gain, offset,
+                   eps, width, n_table_rows, err);
+    } else if (dtype == THN_BF16) {
+        if (smem > 32 * 1024)
+            cudaFuncSetAttribute(embed_norm_kernel<__nv_bfloat16>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+        thn_launch(embed_norm_kernel<__nv_bfloat16>, rows, kThreads, smem, stream, out, copy, (const __nv_bfloat16*)table, tokens,
+                   gain, offset, eps, width, n_table_rows, err);
+    } else {
+        THN_CHECK_ARG(false, "embed_norm: unknown dtype %d", dtype);
+    }
+    return thn_launch_status("embed_norm");
 }
 
 // o float32 [rows, n_heads, size]; gate of the activation type, row stride gate_stride

@@ -5,6 +5,7 @@ engine/engine.py:1101-1121)."""
 
 from __future__ import annotations
 
+from dataclasses import replace
 from typing import Dict, Iterable, List, Optional
 
 import torch
@@ -41,6 +42,7 @@ class DecoderModel:
         self.final_norm = part_class("norm", plan.final_norm.kind)(plan.final_norm, runtime)
         self.head = part_class("head", plan.head.kind)(plan.head, runtime)
         self.vocab_size = plan.vocab_size
+        self.adds_start = any(entry.adds_start for entry in plan.schedule)
         runtime.tensors = {}   # parts hold what they need; fused copies replace the originals
 
     # ------------------------------------------------------------------ construction
@@ -96,9 +98,16 @@ class DecoderModel:
     def hidden(self, tokens: torch.Tensor, ctx: StepContext):
         """All scheduled layers over the step's rows; returns the residual stream and the
         last branch output that has not been added yet."""
-        h = self.embedding.forward(tokens, ctx.err, ctx.rows, ctx.cache)
+        ctx.tokens = tokens
+        start: Optional[torch.Tensor] = None
+        if self.adds_start:
+            h, start = self.embedding.forward_kept(tokens, ctx.err, ctx.rows, ctx.cache)
+        else:
+            h = self.embedding.forward(tokens, ctx.err, ctx.rows, ctx.cache)
         d: Optional[torch.Tensor] = None
         for entry in self.plan.schedule:
+            if entry.adds_start:
+                d = replace(d, add_rows=start) if isinstance(d, Branch) else Branch(d, add_rows=start)
             h, d = self.layers[entry.layer].forward(h, d, ctx, entry)
         return h, d
 
@@ -113,14 +122,11 @@ class DecoderModel:
             if rows is not None:
                 h, y = ops.gather_rows(h, rows), ops.gather_rows(y, rows)
             return self.head.forward(self.final_norm.stream_norm(h, d.write.write.numel(), y=y, written=d.write)[1], err)
-        if isinstance(d, Branch) and (d.second is not None or d.factor != 1.0):
-            # two sublayers side by side, or a factor on the add: the norm takes the branch whole
-            post = d.norm
+        if isinstance(d, Branch) and not d.plain:
+            # two sublayers side by side, or factors on the add: the norm takes the branch whole
             if rows is not None:
-                d = Branch(ops.gather_rows(d.tensor, rows), d.norm,
-                           ops.gather_rows(d.second, rows) if d.second is not None else None, d.factor)
-                h = ops.gather_rows(h, rows)
-            return self.head.forward(self.final_norm.add_forward(h, d, post=post), err)
+                d, h = d.at(rows), ops.gather_rows(h, rows)
+            return self.head.forward(self.final_norm.add_forward(h, d, post=d.norm), err)
         if isinstance(d, Branch):        # a branch that passes a norm of its own before the add
             d, post = d.tensor, d.norm
         if rows is not None:

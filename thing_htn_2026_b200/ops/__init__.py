@@ -57,8 +57,14 @@ _SIGNATURES = {
     "thn_attention_generic": [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int,
                               c_int, c_int, c_int, c_int, c_float, c_int, c_int, c_int, c_int, c_float, c_float, c_int,
                               c_void_p, c_int, c_void_p, c_void_p],
-    "thn_residual_norm": [c_void_p, c_void_p, c_void_p, c_void_p, c_float, c_void_p, c_void_p, c_float, c_float, c_int,
-                          c_void_p, c_void_p, c_float, c_float, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p],
+    "thn_residual_norm": [c_void_p, c_void_p, c_void_p, c_void_p, c_float, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
+                          c_void_p, c_void_p, c_float, c_float, c_int, c_void_p, c_void_p, c_float, c_float, c_int, c_int,
+                          c_int, c_int, c_int, c_int, c_void_p],
+    "thn_embed_norm": [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_float, c_float, c_int, c_int, c_int, c_int,
+                       c_void_p, c_void_p],
+    "thn_token_gate": [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p],
+    "thn_token_gate_product_bf16": [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int,
+                                    c_void_p, c_void_p],
     "thn_gated_head_norm": [c_void_p, c_void_p, c_void_p, c_longlong, c_void_p, c_float, c_int, c_int, c_int, c_int,
                             c_int, c_longlong, c_float, c_int, c_void_p],
     "thn_hyper_norm": [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_float,
@@ -99,7 +105,8 @@ _SIGNATURES = {
     "thn_routed_clamped_glu": [c_void_p, c_void_p, c_void_p, c_void_p, c_longlong, c_int, c_int, c_int, c_int, c_float,
                                c_float, c_float, c_float, c_int, c_int, c_void_p],
     "thn_logistic_gate": [c_void_p, c_void_p, c_void_p, c_longlong, c_int, c_int, c_int, c_int, c_void_p],
-    "thn_latent_norm": [c_void_p, c_void_p, c_longlong, c_void_p, c_float, c_int, c_int, c_int, c_void_p],
+    "thn_latent_norm": [c_void_p, c_longlong, c_void_p, c_int, c_void_p, c_longlong, c_void_p, c_int, c_void_p, c_longlong,
+                        c_float, c_int, c_int, c_void_p],
     "thn_latent_assemble": [c_void_p, c_void_p, c_longlong, c_void_p, c_longlong, c_void_p, c_void_p, c_void_p, c_int,
                             c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int,
                             c_int, c_int, c_void_p, c_void_p],
@@ -524,14 +531,31 @@ class Gain:
 STREAM_AS_IS = Gain(None, 0.0, 1.0, None, "as_is")
 
 
+@dataclass
+class ScaledPair:
+    """Sublayer outputs that are added to the stream entry by entry times a factor (layer scale):
+    ``scale1 * first + scale2 * second``; ``second`` may be None.  The factors are float32 [width]."""
+
+    first: torch.Tensor
+    scale1: torch.Tensor
+    second: Optional[torch.Tensor] = None
+    scale2: Optional[torch.Tensor] = None
+
+    def at(self, rows: torch.Tensor) -> "ScaledPair":
+        return ScaledPair(gather_rows(self.first, rows), self.scale1,
+                          None if self.second is None else gather_rows(self.second, rows), self.scale2)
+
+
 def residual_norm(h: Optional[torch.Tensor], d: Optional[torch.Tensor], post: Optional[Gain], gain: Optional[Gain],
-                  dtype: torch.dtype, d2: Optional[torch.Tensor] = None,
-                  mult: float = 1.0) -> Tuple[torch.Tensor, Optional[torch.Tensor]]:
+                  dtype: torch.dtype, d2: Optional[torch.Tensor] = None, mult: float = 1.0,
+                  scaled: Optional[ScaledPair] = None,
+                  add_rows: Optional[torch.Tensor] = None) -> Tuple[torch.Tensor, Optional[torch.Tensor]]:
     """Norms around a residual stream ``h`` kept in float32 beside activations of ``dtype``:
-    ``h <- h + mult * post(d + d2)`` in place (``post`` None: the branch is added as it is; ``d2``
-    None: one branch; ``h`` None: the stream starts as that), then ``y = gain(h)`` of ``dtype``
-    (``gain`` None: no y; ``STREAM_AS_IS``: y is h rounded).  See :class:`Gain` for the norms.
-    Returns ``(h, y)``."""
+    ``h <- h + scaled + mult * post(d + d2) + add_rows`` in place (``post`` None: the branch is added as it
+    is; ``d2`` None: one output; ``scaled``: outputs with a factor per entry, see :class:`ScaledPair`;
+    ``add_rows``: rows of float32; ``d`` None: no branch; ``h`` None: the stream starts as the branch),
+    then ``y = gain(h)`` of ``dtype`` (``gain`` None: no y; ``STREAM_AS_IS``: y is h rounded).  See
+    :class:`Gain` for the norms.  Returns ``(h, y)``."""
     if d is None and h is None:
         raise KernelError("residual_norm: neither a stream nor a branch")
     h_is_new = h is None
@@ -560,13 +584,78 @@ def residual_norm(h: Optional[torch.Tensor], d: Optional[torch.Tensor], post: Op
                 _need(t, f"residual_norm {what} {name}", torch.float32)
                 if t.shape[0] != width:
                     raise KernelError(f"residual_norm: {what} {name} has {t.shape[0]} entries, rows have {width}")
+    first = second = scale1 = scale2 = None
+    if scaled is not None:
+        first, scale1, second, scale2 = scaled.first, scaled.scale1, scaled.second, scaled.scale2
+        for t, s in ((first, scale1), (second, scale2)) if second is not None else ((first, scale1),):
+            _need(t, "residual_norm scaled output", dtype)
+            _need(s, "residual_norm scale", torch.float32)
+            if tuple(t.shape) != tuple(h.shape) or s.shape[0] != width:
+                raise KernelError(f"residual_norm: scaled output {tuple(t.shape)} with {s.shape[0]} factors, h {tuple(h.shape)}")
+        scale2 = scale2 if second is not None else None
+    if add_rows is not None:
+        _need(add_rows, "residual_norm rows to add", torch.float32)
+        if tuple(add_rows.shape) != tuple(h.shape):
+            raise KernelError(f"residual_norm: rows to add {tuple(add_rows.shape)}, h {tuple(h.shape)}")
     y = torch.empty(h.shape, dtype=dtype, device=h.device) if gain is not None else None
-    _call("thn_residual_norm", _ptr(y), _ptr(h), _ptr(d), _ptr(d2), float(mult), _ptr(post.weight) if post else None,
+    _call("thn_residual_norm", _ptr(y), _ptr(h), _ptr(d), _ptr(d2), float(mult), _ptr(first), _ptr(scale1), _ptr(second),
+          _ptr(scale2), _ptr(add_rows), _ptr(post.weight) if post else None,
           _ptr(post.bias) if post else None, float(post.offset) if post else 0.0, float(post.eps) if post else 1.0,
           NORM_KINDS[post.kind] if post else 0, _ptr(gain.weight) if gain else None, _ptr(gain.bias) if gain else None,
           float(gain.offset) if gain else 0.0, float(gain.eps) if gain else 1.0, NORM_KINDS[gain.kind] if gain else 0,
           int(gain.groups) if gain else 1, rows, width, int(h_is_new), DTYPE_CODE[dtype], _stream())
     return h, y
+
+
+def embed_norm(table: torch.Tensor, tokens: torch.Tensor, gain: Gain, err: Optional[torch.Tensor] = None,
+               copy: bool = False) -> Tuple[torch.Tensor, Optional[torch.Tensor]]:
+    """Token rows that pass an RMS norm as they start a float32 residual stream: ``gain(table[token])``.
+    With ``copy`` the rows are written twice (the stream is updated in place; the copy stays as it is).
+    Returns (stream, copy or None)."""
+    _need(table, "embed_norm table")
+    _need(tokens, "embed_norm tokens", torch.int32)
+    _need(gain.weight, "embed_norm gain", torch.float32)
+    width = table.shape[1]
+    if gain.kind != "rms" or gain.groups != 1 or gain.bias is not None or gain.weight.shape[0] != width:
+        raise KernelError(f"embed_norm: an RMS norm over rows of {width} is needed, not {gain.kind} in {gain.groups} groups of "
+                          f"{gain.weight.shape[0]} gains")
+    out = torch.empty((tokens.shape[0], width), dtype=torch.float32, device=table.device)
+    kept = torch.empty_like(out) if copy else None
+    _call("thn_embed_norm", _ptr(out), _ptr(kept), _ptr(table), _ptr(tokens), _ptr(gain.weight), float(gain.offset),
+          float(gain.eps), tokens.shape[0], width, table.shape[0], _code(table, "embed_norm"), _ptr(err), _stream())
+    return out, kept
+
+
+# Steps of at most this many rows compute a token gate's product in this library's kernel, with the gate behind it.
+TOKEN_GATE_FUSED_ROWS = 16
+
+
+def token_gate(x: torch.Tensor, weight: torch.Tensor, table: torch.Tensor, tokens: torch.Tensor, column: int,
+               err: Optional[torch.Tensor] = None, fused: Optional[bool] = None) -> torch.Tensor:
+    """``gelu(x weight^T) * table[token, column : column + dim]`` with the tanh form of gelu and ``dim`` the
+    weight's rows -> [rows, dim] of the activation type.  One kernel for few rows in bfloat16 (``fused``
+    overrides the choice), a product and a kernel behind it otherwise."""
+    _need(x, "token_gate x")
+    _need(weight, "token_gate weight", x.dtype)
+    _need(table, "token_gate table", x.dtype)
+    _need(tokens, "token_gate tokens", torch.int32)
+    dim, width = weight.shape
+    if x.shape[1] != width or tokens.shape[0] != x.shape[0] or column < 0 or column + dim > table.shape[1]:
+        raise KernelError(f"token_gate: x {tuple(x.shape)}, weight {tuple(weight.shape)}, {tokens.shape[0]} tokens, columns from "
+                          f"{column} of a table {tuple(table.shape)}")
+    can = x.dtype == torch.bfloat16 and width % 8 == 0 and (x.data_ptr() | weight.data_ptr()) % 16 == 0
+    if fused and not can:
+        raise KernelError("token_gate: the kernel with the product takes aligned bfloat16 rows of a multiple of eight entries")
+    if can and (fused or (fused is None and x.shape[0] <= TOKEN_GATE_FUSED_ROWS)):
+        out = torch.empty((x.shape[0], dim), dtype=x.dtype, device=x.device)
+        _call("thn_token_gate_product_bf16", _ptr(out), _ptr(x), _ptr(weight), _ptr(table), _ptr(tokens), x.shape[0], width, dim,
+              table.shape[1], column, table.shape[0], _ptr(err), _stream())
+        return out
+    z = linear(x, weight, err=err)
+    out = torch.empty_like(z)
+    _call("thn_token_gate", _ptr(out), _ptr(z), _ptr(table), _ptr(tokens), z.shape[0], dim, table.shape[1], column,
+          table.shape[0], _code(x, "token_gate"), _ptr(err), _stream())
+    return out
 
 
 GATE_KINDS = {"silu": 0, "logistic": 1}
@@ -1273,32 +1362,41 @@ def delta_rule(proj: torch.Tensor, conv_w: torch.Tensor, a_log: torch.Tensor, dt
 # ------------------------------------------------------------------ latent attention
 
 
-def latent_norm(proj: torch.Tensor, offset: int, rank: int, gain: torch.Tensor, eps: float) -> torch.Tensor:
+def latent_norm(proj: torch.Tensor, offset: int, rank: int, gain: torch.Tensor, eps: float,
+                second: Optional[Tuple[int, int, torch.Tensor]] = None):
     """RMS norm of the ``rank`` entries from column ``offset`` of every projected row, times
     ``gain`` (float32 [rank]) -> [rows, rank] of the rows' type: the latent that the
-    up-projection reads."""
+    up-projection reads.  ``second``: (offset, rank, gain) of another latent of the same rows, normalised
+    in the same launch; the result is then the pair."""
     _need(proj, "latent_norm proj")
-    _need(gain, "latent_norm gain", torch.float32)
-    if gain.shape[0] != rank or offset + rank > proj.shape[1]:
-        raise KernelError(f"latent_norm: {rank} entries from column {offset} of rows of {proj.shape[1]}, gain {tuple(gain.shape)}")
-    out = torch.empty((proj.shape[0], rank), dtype=proj.dtype, device=proj.device)
-    _call("thn_latent_norm", _ptr(out), proj.data_ptr() + offset * proj.element_size(), proj.shape[1], _ptr(gain),
-          float(eps), proj.shape[0], rank, _code(proj, "latent_norm"), _stream())
-    return out
+    outs, parts = [], [(offset, rank, gain)] + ([second] if second is not None else [])
+    for at, n, g in parts:
+        _need(g, "latent_norm gain", torch.float32)
+        if g.shape[0] != n or at < 0 or at + n > proj.shape[1]:
+            raise KernelError(f"latent_norm: {n} entries from column {at} of rows of {proj.shape[1]}, gain {tuple(g.shape)}")
+        outs.append(torch.empty((proj.shape[0], n), dtype=proj.dtype, device=proj.device))
+    at2, n2, g2 = parts[1] if second is not None else (0, 0, None)
+    _call("thn_latent_norm", _ptr(outs[0]), offset, _ptr(gain), rank, _ptr(outs[1]) if second is not None else None, at2, _ptr(g2),
+          n2, _ptr(proj), proj.shape[1], float(eps), proj.shape[0], _code(proj, "latent_norm"), _stream())
+    return outs[0] if second is None else (outs[0], outs[1])
 
 
 def latent_assemble(proj: torch.Tensor, q_offset: int, shared_offset: int, up: torch.Tensor,
                     rotary: Optional[RotaryTables], rows: StepRows, kv: KVView, n_heads: int, plain: int, rot: int,
-                    err: torch.Tensor, value_dim: Optional[int] = None) -> torch.Tensor:
+                    err: torch.Tensor, value_dim: Optional[int] = None, q_rows: Optional[torch.Tensor] = None) -> torch.Tensor:
     """Queries and cache entries of latent attention.  ``proj`` rows hold the queries
     ``[heads][plain | rot]`` from column ``q_offset`` and one shared key part of ``rot`` entries
     from column ``shared_offset``; ``up`` [rows, heads * plain + heads * value] is the
     up-projection of the normalised latent.  The ``rot`` parts are rotated by the rows' positions
     (pairs as ``rotary.layout`` says); the cache gets per head the key ``[plain | rotated shared part]`` and the
     value.  ``value_dim`` (default: the cache's value size) is the size of a value in ``up``; a
-    cache whose values are wider gets zeros behind them.  Returns the queries
+    cache whose values are wider gets zeros behind them.  ``q_rows``: the queries come from rows of their
+    own instead of ``proj``, from column ``q_offset`` of them.  Returns the queries
     [rows, heads * (plain + rot)]."""
     _need(proj, "latent_assemble proj")
+    q_rows = proj if q_rows is None else _need(q_rows, "latent_assemble queries", proj.dtype)
+    if q_rows.shape[0] != proj.shape[0] or q_offset + n_heads * (plain + rot) > q_rows.shape[1]:
+        raise KernelError(f"latent_assemble: query rows {tuple(q_rows.shape)} hold no {n_heads} heads of {plain} + {rot}")
     _need(up, "latent_assemble up", proj.dtype)
     if kv.storage.dtype != proj.dtype or kv.n_kv != n_heads or kv.head_dim != plain + rot:
         raise KernelError(f"latent_assemble: the cache entry ({kv.n_kv} heads of {kv.head_dim}, {kv.storage.dtype}) does "
@@ -1312,7 +1410,7 @@ def latent_assemble(proj: torch.Tensor, q_offset: int, shared_offset: int, up: t
         raise KernelError("latent_assemble: the rotated part needs tables of its size")
     q = torch.empty((rows.n_rows, n_heads * (plain + rot)), dtype=proj.dtype, device=proj.device)
     size = proj.element_size()
-    _call("thn_latent_assemble", _ptr(q), proj.data_ptr() + q_offset * size, proj.shape[1],
+    _call("thn_latent_assemble", _ptr(q), q_rows.data_ptr() + q_offset * size, q_rows.shape[1],
           proj.data_ptr() + shared_offset * size, proj.shape[1], _ptr(up), _ptr(rotary.cos) if rot else None,
           _ptr(rotary.sin) if rot else None, rotary.cos.shape[0] if rot else 0, _ptr(rows.row_slot), _ptr(rows.row_pos),
           _ptr(kv.storage), _ptr(kv.block_table), kv.block_table.shape[1], kv.page_size, rows.n_rows, n_heads, plain, rot,

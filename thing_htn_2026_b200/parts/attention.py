@@ -34,6 +34,12 @@ float32.  ``kv`` "own" (default) or "shared": a "shared" mixer has no key and va
 at all (no ``k_proj`` and ``v_proj`` tensors); every schedule entry that runs it reads the cache
 that another layer wrote (``writes_cache=False``), with its own queries, scale, mask and score
 shaping.
+
+``biases``: the projections among "q", "k", "v" that have one, added in the product (tensors ``q_bias``,
+...).  ``sinks``: a term in the softmax's denominator that has no key and no value, "learned" (``sink``, a
+number per head) or a constant for every head (0.0: one is added to the sum of exponentials).  ``gate``
+"head": a head's output is multiplied by ``logistic(W_g x)``, one number per head (``g_proj``), ahead of the
+output projection; the gate's rows ride in the same product as q, k and v.
 """
 
 from __future__ import annotations
@@ -46,6 +52,7 @@ from .. import ops
 from ..cache.sequence_cache import CacheNeed, KVSpec
 from ..config.base import PartSpec, ScheduleEntry
 from ..weights.loader import GAIN, MATRIX, TensorSpec
+from .fused import cat_bias, pad_rows
 from .registry import part_class, register_part
 from .runtime import HostBatch, Runtime, StepContext
 
@@ -62,6 +69,13 @@ class Attention:
             specs.append(TensorSpec(spec.tensors["k_proj"], (n_kv * d, hidden), MATRIX))
             if p.get("values", "projection") == "projection":
                 specs.append(TensorSpec(spec.tensors["v_proj"], (n_kv * dv, hidden), MATRIX))
+        for name, size in (("q", n_q * d), ("k", n_kv * d), ("v", n_kv * dv)):
+            if name in (p.get("biases") or ()):
+                specs.append(TensorSpec(spec.tensors[name + "_bias"], (size,), MATRIX, init="small_normal"))
+        if p.get("sinks") == "learned":
+            specs.append(TensorSpec(spec.tensors["sink"], (n_q,), GAIN, init="sink"))
+        if p.get("gate"):
+            specs.append(TensorSpec(spec.tensors["g_proj"], (n_q, hidden), MATRIX))
         specs.append(TensorSpec(spec.tensors["o_proj"], (hidden, n_q * dv), MATRIX))
         if p.get("qk_norm_eps") is not None:
             whole = p.get("qk_norm_scope", "head") == "projection"
@@ -94,12 +108,25 @@ class Attention:
         self.shared_kv = p.get("kv", "own") == "shared"
         if self.shared_kv and (p.get("qk_norm_eps") is not None or p.get("position") is not None):
             raise ValueError("attention: a mixer without keys of its own has no q/k norm and no rotation here")
-        projections = [runtime.tensor(spec, "q_proj")]
-        if not self.shared_kv:
-            projections.append(runtime.tensor(spec, "k_proj"))
-            if not self.values_are_keys:
-                projections.append(runtime.tensor(spec, "v_proj"))
-        self.w_qkv = torch.cat(projections, dim=0).contiguous() if len(projections) > 1 else projections[0]
+        names = ["q"] if self.shared_kv else ["q", "k"] if self.values_are_keys else ["q", "k", "v"]
+        biases = tuple(p.get("biases") or ())
+        if set(biases) - set(names):
+            raise ValueError(f"attention: biases {biases} of projections among {names}")
+        rows = [(runtime.tensor(spec, n + "_proj"), runtime.tensor(spec, n + "_bias") if n in biases else None) for n in names]
+        if p.get("gate") not in (None, "head"):
+            raise ValueError(f"attention: gate {p.get('gate')!r} is neither None nor 'head'")
+        self.gated = p.get("gate") == "head"
+        self.gate_offset = sum(w.shape[0] for w, _ in rows)
+        if self.gated:
+            rows.append((pad_rows(runtime.tensor(spec, "g_proj"), self.gate_offset), None))
+        self.w_qkv = torch.cat([w for w, _ in rows], dim=0).contiguous() if len(rows) > 1 else rows[0][0]
+        self.b_qkv = cat_bias(rows)
+        sinks = p.get("sinks")
+        self.sinks = None
+        if sinks == "learned":
+            self.sinks = runtime.tensor(spec, "sink").to(torch.float32).contiguous()
+        elif sinks is not None:
+            self.sinks = torch.full((self.n_q,), float(sinks), dtype=torch.float32, device=runtime.device)
         temp = p.get("q_temp")
         self.shape = ops.ScoreShape(float(p.get("softcap") or 0.0), float(temp["coef"]) if temp else 0.0,
                                     int(temp["every"]) if temp else 0)
@@ -119,7 +146,7 @@ class Attention:
         # The per-head kernel (and the kernel that fuses it with single-token attention) takes the
         # defaults; every other variant is prepared by the general kernel.
         self.general = (self.norm_scope == "projection" or self.values_are_keys
-                        or p.get("prepare") == "float32" or self.value_dim != self.head_dim
+                        or p.get("prepare") == "float32" or self.value_dim != self.head_dim or self.gated
                         or (self.position is not None and getattr(self.position, "layout", "half") != "half"))
         if self.general and self.eps is not None:
             self.q_gain, self.k_gain = self.q_gain.float().contiguous(), self.k_gain.float().contiguous()
@@ -142,6 +169,11 @@ class Attention:
             out[f"row_tiles/{size}/row0"], out[f"row_tiles/{size}/rows"] = ops.row_tiles_of(
                 batch.counts, batch.held, size)
 
+    def _out(self, a: torch.Tensor, proj: torch.Tensor, ctx: StepContext) -> torch.Tensor:
+        if self.gated:
+            a = ops.logistic_gate(a, proj, self.gate_offset, self.value_dim)
+        return ops.linear(a, self.w_o, err=ctx.err)
+
     def forward(self, x: torch.Tensor, ctx: StepContext, entry: ScheduleEntry) -> torch.Tensor:
         kv = ctx.cache.kv_view(entry.cache)
         tiles = None
@@ -150,15 +182,17 @@ class Attention:
             row0 = ctx.inputs.get(f"row_tiles/{size}/row0") if size else None
             if row0 is not None:
                 tiles = ops.RowTiles(row0, ctx.inputs[f"row_tiles/{size}/rows"], row0.shape[0], size)
-        qkv = ops.linear(x, self.w_qkv, err=ctx.err)
+        qkv = ops.linear(x, self.w_qkv, err=ctx.err, bias=self.b_qkv)
         if self.shared_kv:
             if entry.writes_cache:
                 raise ValueError("attention: a mixer without keys of its own cannot write a cache")
             # the projected rows are the queries: nothing to normalise, rotate or store
-            a = ops.attention(qkv, ctx.rows, kv, self.n_q, self.scale, self.window, ctx.err, tiles, self.keep_first,
-                              self.chunk, self.exact_weights, self.shape)
-            return ops.linear(a, self.w_o, err=ctx.err)
-        if self.general or self.keep_first or self.chunk or self.exact_weights or self.shape.active:
+            q = qkv[:, :self.gate_offset].contiguous() if self.gated else qkv
+            a = ops.attention(q, ctx.rows, kv, self.n_q, self.scale, self.window, ctx.err, tiles, self.keep_first,
+                              self.chunk, self.exact_weights, self.shape, self.sinks)
+            return self._out(a, qkv, ctx)
+        if (self.general or self.keep_first or self.chunk or self.exact_weights or self.shape.active
+                or self.sinks is not None):
             rotary = self.position.tables() if self.position is not None else None
             if self.general:
                 q = ops.qk_prepare(qkv, self.q_gain, self.k_gain, self.norm_scope, self.eps or 1.0, rotary, ctx.rows, kv,
@@ -167,8 +201,8 @@ class Attention:
                 q = ops.qk_norm_rope_cache(qkv, self.q_gain, self.k_gain, self.eps if self.eps is not None else 1.0,
                                            rotary, ctx.rows, kv, self.n_q, entry.writes_cache, ctx.err)
             a = ops.attention(q, ctx.rows, kv, self.n_q, self.scale, self.window, ctx.err, tiles, self.keep_first,
-                              self.chunk, self.exact_weights, self.shape)
-            return ops.linear(a, self.w_o, err=ctx.err)
+                              self.chunk, self.exact_weights, self.shape, self.sinks)
+            return self._out(a, qkv, ctx)
         a = ops.qkv_attention(qkv, self.q_gain, self.k_gain, self.eps if self.eps is not None else 1.0,
                               self.position.tables() if self.position is not None else None,
                               ctx.rows, kv, self.n_q, self.scale, self.window, entry.writes_cache, ctx.err, tiles)

@@ -23,7 +23,10 @@ feed-forward half may be absent.  The pending output again travels as a :class:`
 ``y = x + factor * (mixer(n) + ffn(n))`` over a float32 stream (``factor`` a parameter of the
 block, default 1; the feed-forward may be absent).  The two outputs travel as one
 :class:`Branch` with its second tensor and its factor, so that "add both, times the factor, into
-the stream, norm of the sum" is one kernel at the next layer's norm or at the model's last.
+the stream, norm of the sum" is one kernel at the next layer's norm or at the model's last.  With
+``layer_scale`` (and the tensors ``mixer_scale`` and, beside a feed-forward, ``ffn_scale``, a vector each)
+it is ``y = x + s * mixer(n) + s' * ffn(n)``, entry by entry.  ``side``: a part that adds something of its own
+behind the sublayers, ``z = y + side(y)`` (:mod:`.side`).
 
 ``hyper_connections``: the residual stream is ``streams`` copies ``X_0 .. X_(s-1)`` in float32,
 all equal to the embedding's row at the start.  A sublayer f with the numbers ``read[s]``,
@@ -116,7 +119,7 @@ class SandwichNormBlock(Block):
             else:                      # the embedding's rows start the float32 stream
                 h, n = self.norm_mixer.start_forward(h)
         elif isinstance(d, Branch):
-            n = self.norm_mixer.add_forward(h, d.tensor, post=d.norm)
+            n = self.norm_mixer.add_forward(h, d.tensor, post=d.norm) if d.plain else self.norm_mixer.add_forward(h, d)
         else:
             n = self.norm_mixer.add_forward(h, d)
         a = Branch(self.mixer.forward(n, ctx, entry), self.post_norm_mixer)
@@ -135,7 +138,7 @@ class BranchNormBlock(Block):
             raise TypeError("branch_norm: the residual stream must start in float32 (an embedding with stream 'float32')")
         if d is None:
             x = self.norm_mixer.read(h)
-        elif isinstance(d, Branch) and d.norm is not None:
+        elif isinstance(d, Branch) and d.norm is not None and d.plain:
             x = d.norm.add_read(h, d.tensor)
         else:
             raise TypeError("branch_norm: a pending branch must name the norm it passes before the add")
@@ -148,11 +151,27 @@ class BranchNormBlock(Block):
 
 @register_part("block", "parallel")
 class ParallelBlock(Block):
-    MEMBERS = {"norm": "norm", "mixer": "mixer", "ffn": "ffn"}
+    MEMBERS = {"norm": "norm", "mixer": "mixer", "ffn": "ffn", "side": "side"}
+
+    @classmethod
+    def tensor_specs(cls, spec: PartSpec) -> List[TensorSpec]:
+        specs = super().tensor_specs(spec)
+        if spec.params.get("layer_scale"):
+            size = int(spec.params["norm"].params["size"])
+            names = ["mixer_scale"] + (["ffn_scale"] if spec.params.get("ffn") is not None else [])
+            specs += [TensorSpec(spec.tensors[name], (size,), GAIN) for name in names]
+        return specs
 
     def __init__(self, spec: PartSpec, runtime: Runtime):
         super().__init__(spec, runtime)
         self.factor = float(spec.params.get("factor", 1.0))
+        self.mixer_scale = self.ffn_scale = None
+        if spec.params.get("layer_scale"):
+            if self.factor != 1.0:
+                raise ValueError("parallel: layer_scale stands instead of a factor")
+            self.mixer_scale = runtime.tensor(spec, "mixer_scale").to(torch.float32).contiguous()
+            if self.ffn is not None:
+                self.ffn_scale = runtime.tensor(spec, "ffn_scale").to(torch.float32).contiguous()
 
     def forward(self, h: torch.Tensor, d, ctx: StepContext, entry: ScheduleEntry):
         if h.dtype != torch.float32:
@@ -165,7 +184,13 @@ class ParallelBlock(Block):
             n = self.norm.add_forward(h, d)
         a = self.mixer.forward(n, ctx, entry)
         f = self.ffn.forward(n, ctx) if self.ffn is not None else None
-        return h, Branch(a, None, f, self.factor)
+        if self.mixer_scale is not None:
+            d = Branch(None, scaled=ops.ScaledPair(a, self.mixer_scale, f, self.ffn_scale))
+        else:
+            d = Branch(a, None, f, self.factor)
+        if self.side is None:
+            return h, d
+        return h, self.side.forward(self.norm.add_read(h, d), ctx)
 
 
 @register_part("block", "hyper_connections")
@@ -210,7 +235,7 @@ class HyperConnectionBlock(Block):
         own = self.numbers["mixer"]
         if d is None:           # the model's first layer: every copy starts as the embedding's row
             X, n = self.norm_mixer.stream_norm(None, self.streams, start=h, read=own.read)
-        elif isinstance(d, Branch) and d.write is not None:
+        elif isinstance(d, Branch) and d.write is not None and d.add_rows is None:
             X, n = self.norm_mixer.stream_norm(h, self.streams, y=d.tensor, written=d.write, read=own.read)
         else:
             raise TypeError("hyper_connections: a pending branch must carry the numbers of its write")

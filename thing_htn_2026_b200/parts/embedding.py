@@ -14,7 +14,9 @@ then the most positions a sequence can have.  ``pairs`` (a mapping ``buckets, mu
 float32 stream only): a row of the tensor ``pairs`` [buckets + 1, hidden] is added for every pair of
 neighbouring tokens, number ``(before * mul_before + token * mul_token) mod buckets``, the last row for
 a sequence's first token.  The token before the first one of a step is per-sequence state
-(``previous_token``, registered through ``sequence_states``).
+(``previous_token``, registered through ``sequence_states``).  ``norm`` (the spec of an RMS norm; float32
+stream only, without a scale, positions or pairs): the token's row passes this norm as it starts the stream.
+``forward_kept`` gives the start of the stream twice, for a model that adds it again later.
 
 The head takes ``scale`` (default 1): a constant factor on the logits."""
 
@@ -27,7 +29,7 @@ import torch
 from .. import ops
 from ..config.base import PartSpec
 from ..weights.loader import MATRIX, TensorSpec
-from .registry import register_part
+from .registry import part_class, register_part
 from .runtime import Runtime
 
 
@@ -41,6 +43,8 @@ class Embedding:
             specs.append(TensorSpec(spec.tensors["pairs"], (int(p["pairs"]["buckets"]) + 1, width), MATRIX))
         if p.get("positions") is not None and p["positions"].get("kind") == "learned":
             specs.append(TensorSpec(spec.tensors["positions"], (int(p["positions"]["size"]), width), MATRIX))
+        if p.get("norm") is not None:
+            specs += part_class("norm", p["norm"].kind).tensor_specs(p["norm"])
         return specs
 
     def __init__(self, spec: PartSpec, runtime: Runtime):
@@ -68,6 +72,11 @@ class Embedding:
             self.pairs = ops.PairTable(runtime.tensor(spec, "pairs"), int(pairs["mul_before"]), int(pairs["mul_token"]))
         if self.pairs is not None and self.frequencies is not None:
             raise ValueError("embedding: pairs go with learned positions or none")
+        self.norm = None
+        if spec.params.get("norm") is not None:
+            if not self.float32_stream or self.scale != 1.0 or positions is not None or pairs is not None:
+                raise ValueError("embedding: a norm needs stream 'float32', and no scale, positions or pairs")
+            self.norm = part_class("norm", spec.params["norm"].kind)(spec.params["norm"], runtime)
 
     def sequence_states(self) -> Dict[str, Tuple[Tuple[int, ...], torch.dtype]]:
         """Per-sequence state by name (shape without the slots, dtype), zeroed when a slot opens."""
@@ -77,6 +86,8 @@ class Embedding:
                 cache=None) -> torch.Tensor:
         """``rows``: the step's rows, for an embedding that adds positions or pairs; ``cache``: the
         sequences' cache, for one that adds pairs or learned positions."""
+        if self.norm is not None:
+            return ops.embed_norm(self.table, tokens, self.norm.as_gain, err)[0]
         if self.pairs is not None or self.positions is not None:
             if rows is None or cache is None:
                 raise ValueError("embedding: pairs or learned positions are added, the step's rows and cache are needed")
@@ -89,6 +100,17 @@ class Embedding:
         if self.float32_stream:
             return ops.gather_rows_scaled(self.table, tokens, self.scale, err)
         return ops.gather_rows(self.table, tokens, err)
+
+
+    def forward_kept(self, tokens: torch.Tensor, err: torch.Tensor, rows: Optional[ops.StepRows] = None,
+                     cache=None) -> Tuple[torch.Tensor, torch.Tensor]:
+        """(the float32 stream's start, the same rows once more)."""
+        if not self.float32_stream:
+            raise ValueError("embedding: the start of a stream can be kept where the stream is float32")
+        if self.norm is not None:
+            return ops.embed_norm(self.table, tokens, self.norm.as_gain, err, copy=True)
+        h = self.forward(tokens, err, rows, cache)
+        return h, h.clone()
 
 
 @register_part("head", "lm_head")

@@ -35,6 +35,13 @@ def cat_bias(pieces: List[Tuple[torch.Tensor, Optional[torch.Tensor]]]) -> Optio
                       for w, b in pieces]).contiguous()
 
 
+def pad_rows(weight: torch.Tensor, ahead: int, multiple: int = 8) -> torch.Tensor:
+    """A weight ``[n, hidden]`` that stands behind ``ahead`` other rows, with rows of zeros appended so that the
+    projected rows are whole 16-byte pieces."""
+    short = -(ahead + weight.shape[0]) % multiple
+    return weight if not short else torch.nn.functional.pad(weight, (0, 0, 0, short))
+
+
 class PhasedMixer:
     """Base of the mixers in three phases.  ``state_base``: the index of this mixer's first state
     tensor in its cache entry (a pair moves the second mixer's behind the first's)."""

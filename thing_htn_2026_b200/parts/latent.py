@@ -17,6 +17,11 @@ i sees j with 0 <= i - j < window.  ``gated`` False leaves the output gate (and 
 ``gate_scope`` "value" (the default): a gate per entry, as above; "head": one number per head,
 ``W_g`` has ``n_heads`` rows and a head's output is multiplied by its gate.
 
+``q_rank``: the queries are read out of a latent of their own, ``q = W_uq (RMSnorm(W_dq x) * w_qnorm)``, with
+the tensors ``q_down`` [q_rank, hidden], ``q_norm`` [q_rank] and ``q_proj`` [heads * (plain + rot), q_rank]; both
+latents are normalised in one launch.  ``sinks`` "learned": the softmax's denominator of head h also
+holds ``exp(sink_h)``, a term without key and value (``sink``, a number per head).
+
 One product gives q, the latent row and the gate (weights concatenated ``[q; dkv; g]``); a
 second one, on the normalised latent, gives every head's unrotated key and value (``[uk; uv]``).
 The cache holds per head the assembled key and the value (a window bounds what a sequence
@@ -37,6 +42,7 @@ from .. import ops
 from ..cache.sequence_cache import PAGE_SIZE, CacheNeed, KVSpec
 from ..config.base import PartSpec, ScheduleEntry
 from ..weights.loader import GAIN, MATRIX, TensorSpec
+from .fused import pad_rows
 from .registry import part_class, register_part
 from .runtime import HostBatch, Runtime, StepContext
 
@@ -52,7 +58,14 @@ class LatentAttention:
     @classmethod
     def tensor_specs(cls, spec: PartSpec) -> List[TensorSpec]:
         hidden, h, d, r, e, c = cls._sizes(spec)
-        specs = [TensorSpec(spec.tensors["q_proj"], (h * (d + r), hidden), MATRIX),
+        q_rank = int(spec.params.get("q_rank") or 0)
+        specs = []
+        if q_rank:
+            specs += [TensorSpec(spec.tensors["q_down"], (q_rank, hidden), MATRIX),
+                      TensorSpec(spec.tensors["q_norm"], (q_rank,), GAIN)]
+        if spec.params.get("sinks"):
+            specs.append(TensorSpec(spec.tensors["sink"], (h,), GAIN, init="sink"))
+        specs += [TensorSpec(spec.tensors["q_proj"], (h * (d + r), q_rank or hidden), MATRIX),
                  TensorSpec(spec.tensors["down_proj"], (c + r, hidden), MATRIX),
                  TensorSpec(spec.tensors["latent_norm"], (c,), GAIN),
                  TensorSpec(spec.tensors["up_k"], (h * d, c), MATRIX),
@@ -84,13 +97,25 @@ class LatentAttention:
                 and ops.lib().thn_attention_mma_supported(key_dim, PAGE_SIZE, self.n_heads, self.n_heads):
             self.out_dim = key_dim
         pad = self.out_dim - self.value_dim
-        parts = [runtime.tensor(spec, "q_proj"), runtime.tensor(spec, "down_proj")]
+        self.q_rank = int(p.get("q_rank") or 0)
+        if p.get("sinks") not in (None, "learned"):
+            raise ValueError(f"latent_attention: sinks {p.get('sinks')!r} are neither None nor 'learned'")
+        self.sinks = runtime.tensor(spec, "sink").to(torch.float32).contiguous() if p.get("sinks") else None
+        # the projected row: the queries (or their latent), the latent with the shared key part, the gate
+        self.latent_offset = self.q_rank or self.n_heads * key_dim
+        self.shared_offset = self.latent_offset + self.rank
+        self.gate_offset = self.shared_offset + self.rot
+        self.w_uq = self.q_gain = None
+        if self.q_rank:
+            self.w_uq = runtime.tensor(spec, "q_proj")
+            self.q_gain = runtime.tensor(spec, "q_norm").to(torch.float32).contiguous()
+        parts = [runtime.tensor(spec, "q_down" if self.q_rank else "q_proj"), runtime.tensor(spec, "down_proj")]
         if self.gated:
             gate = runtime.tensor(spec, "g_proj")
             if pad and not self.head_gate:
                 gate = torch.nn.functional.pad(gate.view(self.n_heads, self.value_dim, hidden), (0, 0, 0, pad))
                 gate = gate.reshape(self.n_heads * self.out_dim, hidden)
-            parts.append(gate)
+            parts.append(pad_rows(gate, self.gate_offset) if self.head_gate else gate)
         self.w_in = torch.cat(parts, dim=0).contiguous()
         self.w_up = torch.cat([runtime.tensor(spec, "up_k"), runtime.tensor(spec, "up_v")], dim=0).contiguous()
         self.w_o = runtime.tensor(spec, "o_proj")
@@ -98,9 +123,6 @@ class LatentAttention:
             self.w_o = torch.nn.functional.pad(self.w_o.view(hidden, self.n_heads, self.value_dim), (0, pad))
             self.w_o = self.w_o.reshape(hidden, self.n_heads * self.out_dim).contiguous()
         self.latent_gain = runtime.tensor(spec, "latent_norm").to(torch.float32).contiguous()
-        self.latent_offset = self.n_heads * (self.plain + self.rot)
-        self.shared_offset = self.latent_offset + self.rank
-        self.gate_offset = self.shared_offset + self.rot
         self.position = None
         position_spec = p.get("position")
         if self.rot:
@@ -135,12 +157,18 @@ class LatentAttention:
             if row0 is not None:
                 tiles = ops.RowTiles(row0, ctx.inputs[f"row_tiles/{size}/rows"], row0.shape[0], size)
         proj = ops.linear(x, self.w_in, err=ctx.err)
-        latent = ops.latent_norm(proj, self.latent_offset, self.rank, self.latent_gain, self.eps)
+        q_rows = None
+        if self.q_rank:
+            q_latent, latent = ops.latent_norm(proj, 0, self.q_rank, self.q_gain, self.eps,
+                                               second=(self.latent_offset, self.rank, self.latent_gain))
+            q_rows = ops.linear(q_latent, self.w_uq, err=ctx.err)
+        else:
+            latent = ops.latent_norm(proj, self.latent_offset, self.rank, self.latent_gain, self.eps)
         up = ops.linear(latent, self.w_up, err=ctx.err)
         q = ops.latent_assemble(proj, 0, self.shared_offset, up, self.position.tables() if self.position else None,
-                                ctx.rows, kv, self.n_heads, self.plain, self.rot, ctx.err, self.value_dim)
+                                ctx.rows, kv, self.n_heads, self.plain, self.rot, ctx.err, self.value_dim, q_rows)
         a = ops.attention(q, ctx.rows, kv, self.n_heads, self.scale, self.window, ctx.err, tiles,
-                          exact_weights=self.exact_weights)
+                          exact_weights=self.exact_weights, sinks=self.sinks)
         if self.gated:
             a = ops.logistic_gate(a, proj, self.gate_offset, self.out_dim if self.head_gate else 1)
         return ops.linear(a, self.w_o, err=ctx.err)

@@ -10,8 +10,9 @@ also takes ``post``: another norm of this kind that the branch's output passes b
 added (norms on both sides of a sublayer), in the same kernel.  ``groups`` (default 1; float32
 stream only): the row is split into that many equal consecutive parts, each divided by its own
 ``sqrt(mean(part^2) + eps)``, and the whole is multiplied by the gain.  ``add_forward`` takes a
-:class:`Branch` as well: its second tensor and its factor are added in the same kernel,
-``h <- h + factor * (d + d')``.  ``gain`` "scalar": the gain is one number (a tensor without
+:class:`Branch` as well: its second tensor, its factor, outputs with a factor per entry and rows to
+add are taken in the same kernel, ``h <- h + (s p + s' p') + factor * post(d + d') + rows``; ``add_read``
+adds such a branch and returns the stream itself, rounded.  ``gain`` "scalar": the gain is one number (a tensor without
 axes) for all coordinates.  ``stream_norm`` serves a residual stream of several copies
 (hyper-connections, :func:`ops.hyper_norm`): the pending write of the sublayer before, the read of
 the next one and this norm of what was read, in one kernel.
@@ -95,14 +96,25 @@ class RMSNorm:
     def add_forward(self, h: torch.Tensor, d, post: Optional["RMSNorm"] = None) -> torch.Tensor:
         if isinstance(d, Branch):       # a branch with a second tensor or a factor (its norm comes as ``post``)
             if not self.float32_stream:
-                raise ops.KernelError("rmsnorm: a branch of two tensors or with a factor needs a float32 stream")
-            return ops.residual_norm(h, d.tensor, post.as_gain if post is not None else None, self.as_gain, self.dtype,
-                                     d2=d.second, mult=d.factor)[1]
+                raise ops.KernelError("rmsnorm: a branch of more than one plain output needs a float32 stream")
+            return self._add_branch(h, d, self.as_gain, post)
         if self.float32_stream:
             return ops.residual_norm(h, d, post.as_gain if post is not None else None, self.as_gain, self.dtype)[1]
         if post is not None or self.offset:
             raise ops.KernelError("rmsnorm: a norm of the branch before the add, or a gain offset, needs a float32 stream")
         return ops.add_rmsnorm(h, d, self.gain, self.eps)
+
+    def _add_branch(self, h: torch.Tensor, d: Branch, gain, post: Optional["RMSNorm"]) -> torch.Tensor:
+        post = post if post is not None else d.norm
+        return ops.residual_norm(h, d.tensor, post.as_gain if post is not None else None, gain, self.dtype, d2=d.second,
+                                 mult=d.factor, scaled=d.scaled, add_rows=d.add_rows)[1]
+
+    def add_read(self, h: torch.Tensor, d: Branch) -> torch.Tensor:
+        """Adds a pending branch to a float32 stream; returns the new stream rounded to the activation
+        type, for a part that reads the stream itself."""
+        if not self.float32_stream:
+            raise ops.KernelError("rmsnorm: reading the stream itself goes with a float32 stream")
+        return self._add_branch(h, d, ops.STREAM_AS_IS, None)
 
     def add_only(self, h: torch.Tensor, d: torch.Tensor) -> None:
         """``h <- h + self(d)`` on a float32 stream, nothing else: this norm as the one a branch

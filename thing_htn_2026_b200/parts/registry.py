@@ -7,7 +7,7 @@ from __future__ import annotations
 
 from typing import Callable, Dict, Tuple
 
-FAMILIES = ("embedding", "mixer", "ffn", "norm", "position", "block", "head")
+FAMILIES = ("embedding", "mixer", "ffn", "norm", "position", "block", "head", "side")
 
 _PARTS: Dict[Tuple[str, str], type] = {}
 
