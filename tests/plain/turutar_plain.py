@@ -133,7 +133,7 @@ def window_attention(ar, h, w, prefix, m, eps):
     k = ar.rb(rms_divide(k, eps) * w[prefix + "k.norm"].to(ar.work)).reshape(T, G, d)
     place = torch.arange(T)
     behind = place[:, None] - place[None, :]
-    visible = (behind >= 0) & (behind < m["mask"]["size"])
+    visible = (behind >= 0) & (behind < m["mask"]["size"] if m.get("mask") else behind >= 0)
     gate = logistic(ar.linear(h, w[prefix + "g"]))
     out = torch.zeros(T, H, d, dtype=ar.work)
     for head in range(H):

@@ -153,3 +153,23 @@ def test_a_futepel_model_written_and_run_from_the_command_line(tmp_path):
     lines = [json.loads(line) for line in run_cli("bench", "--random-config", "futepel-tiny", "--shapes", "2x16x8",
                                                   "--repeats", "1")]
     assert lines[0]["shape"] == "2x16x8" and lines[0]["tok_per_s"] > 0
+
+
+def test_a_turutar_model_written_and_run_from_the_command_line(tmp_path):
+    """The same for the seventh architecture, with both mixers, looped layers, token rows and a layer without
+    a feed-forward: a named configuration written as a folder, read back by ``generate``, the entry point's
+    tokens, and ``bench``."""
+    from thing_htn_2026_b200 import Engine, cli
+    folder = str(tmp_path / "turutar")
+    assert run_cli("random-model", "--random-config", "turutar-tiny", "--seed", "4", "--out", folder, "--dtype",
+                   "bfloat16") == [folder]
+    with open(os.path.join(folder, "config.json")) as handle:
+        assert json.load(handle)["architecture"] == "Turutar"
+    printed = [json.loads(line) for line in run_cli("generate", "--model", folder, "--prompt-lens", "3,70,21", "--seed", "5",
+                                                    "--max-new-tokens", "9", "--dtype", "float32")]
+    engine = Engine(folder, dtype="float32")
+    steps = list(engine.generate(cli.make_prompts_of([3, 70, 21], engine.model.vocab_size, 5), 9))
+    assert [p["tokens"] for p in printed] == [[step[j] for step in steps] for j in range(3)]
+    lines = [json.loads(line) for line in run_cli("bench", "--random-config", "turutar-tiny", "--shapes", "2x16x8",
+                                                  "--repeats", "1")]
+    assert lines[0]["shape"] == "2x16x8" and lines[0]["tok_per_s"] > 0

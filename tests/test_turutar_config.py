@@ -214,3 +214,38 @@ def test_a_later_pass_adds_the_start_once():
     start = plain.embed(w, data, torch.tensor(toks), torch.float64)
     after = plain.model_forward(None, toks, torch.float64, (data, w))[1]
     assert [round((a / start).mean().item(), 9) for a in after] == [1.0, 1.0, 2.0, 2.0, 3.0, 3.0, 3.0]
+
+
+# ----------------------------------------------------------------------------- what comparisons with it show
+
+
+@pytest.fixture(scope="module")
+def folder(tmp_path_factory):
+    return tiny.write_model(str(tmp_path_factory.mktemp("turutar") / "a"), "a")
+
+
+def changed(folder, change):
+    """Exact logits of 150 tokens with a mistake planted in the plain implementation, and without."""
+    config, w = plain.read_model(folder)
+    toks = tiny.tokens("a", 150, 77)
+    right = plain.model_forward(None, toks, torch.float64, (config, w))[0].numpy()
+    change(config, w)
+    difference = plain.model_forward(None, toks, torch.float64, (config, w))[0].numpy() - right
+    return (difference - difference.mean(axis=1, keepdims=True)).std(axis=1)
+
+
+@pytest.mark.parametrize("what, change", [
+    ("window one longer", lambda c, w: c["layers"][0]["mixer"]["mask"].update(size=21)),
+    ("window one shorter", lambda c, w: c["layers"][2]["mixer"]["mask"].update(size=32)),
+    ("sinks left out", lambda c, w: w.update({"l1.mix.sink": torch.full((3,), -100.0)})),
+    ("biases left out", lambda c, w: w.update({"l0.mix.k.b": torch.zeros(24)})),
+    ("one pass fewer", lambda c, w: c["loop"].update(times=1)),
+    ("loop from the first layer", lambda c, w: c["loop"].update(start=0)),
+    ("another layer's columns", lambda c, w: w.update({"side.embed": w["side.embed"].roll(10, 1)})),
+    ("layer scales swapped", lambda c, w: w.update({"l0.ls1": w["l0.ls2"], "l0.ls2": w["l0.ls1"]})),
+    ("gate of another head", lambda c, w: w.update({"l0.mix.g": w["l0.mix.g"].roll(1, 0)})),
+    ("another limit", lambda c, w: c["layers"][0]["mlp"].update(limit=0.7)),
+])
+def test_what_the_comparisons_would_show(folder, what, change):
+    """Mistakes planted in the plain implementation move the logits far beyond the tolerances of the comparisons on the device."""
+    assert changed(folder, change)[60:].max() > 1e-2, what

@@ -80,7 +80,7 @@ def config_json(name):
 def write_model(folder, name, dtype=torch.bfloat16):
     """Random weights through the library's random-weights mode (stored in bfloat16, as served models
     are), with matrices wide enough that attention weights are far from uniform, layer scales of either
-    sign, and biases and norms inside the mixers of the order of what they stand beside."""
+    sign, and biases, sinks and norms inside the mixers of the order of what they stand beside."""
     from thing_htn_2026_b200.config import config_from_dict
     from thing_htn_2026_b200.weights import random_tensors_cpu
     from thing_htn_2026_b200.weights.safetensors_io import write_safetensors
@@ -92,6 +92,8 @@ def write_model(folder, name, dtype=torch.bfloat16):
             tensors[key] = (torch.randn(tensors[key].shape, generator=g) * 0.5 + 0.4).to(dtype)
         elif key.endswith((".q.b", ".k.b")):
             tensors[key] = (torch.randn(tensors[key].shape, generator=g) * 0.6).to(dtype)
+        elif key.endswith(".sink"):
+            tensors[key] = (torch.randn(tensors[key].shape, generator=g) + 3.5).to(dtype)
         elif key == "embed":
             tensors[key] = (torch.randn(tensors[key].shape, generator=g) * torch.rand(tensors[key].shape[0], 1, generator=g)).to(dtype)
     os.makedirs(folder, exist_ok=True)
