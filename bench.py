@@ -39,7 +39,11 @@ experts weighted at their output) beside a Bunudra decoder of the same width, de
 experts, its closest relative here.  ``--design futepel`` measures the Futepel decoder
 (``futepel-w2048``, ``futepel-w4096``: state-space duality, time mixing and latent attention over a plain
 float32 stream, dense squared-relu and routed feed-forwards) beside a Bunudra decoder of the same
-width, depth, latent attention and feed-forward weights.  The default run is untouched by all five.
+width, depth, latent attention and feed-forward weights.  ``--design turutar`` measures the Turutar
+decoder (``turutar-w2048``, ``turutar-w4096``: windowed attention with an added one and latent attention with
+sinks, parallel sublayers with layer scale, four of eight layers run twice, token rows beside every layer)
+beside a Lanilix decoder of attention layers with the same width, heads, windows and feed-forward, one
+for every execution of a layer.  The default run is untouched by all six.
 """
 
 from __future__ import annotations
@@ -1536,6 +1540,174 @@ def futepel_kernel_table(torch, fut, peak, batch, context):
     return table.finished()
 
 
+TURUTAR_SIZES = ("turutar-w2048", "turutar-w4096")
+
+
+def lanilix_like_turutar(tur):
+    """A Lanilix config.json of the same width, feed-forward and vocabulary as a Turutar configuration, with
+    an attention layer for every execution of one (those of later passes over a loop use the first one's
+    weights): the same heads and window for a windowed layer, for a latent one as many heads of the keys'
+    size over all keys."""
+    from thing_htn_2026_b200.config import config_from_dict
+    layers, first = [], {}
+    for i, entry in enumerate(config_from_dict(tur).plan().schedule):
+        layer = tur["layers"][entry.layer]
+        m = layer["mixer"]
+        if layer["type"] == "attention":
+            heads, kv_heads, d, mask = m["heads"], m["kv_heads"], m["dim"], {"size": m["mask"]["size"], "keep_first": 0}
+        else:
+            heads, kv_heads, d, mask = m["heads"], m["heads"], m["dim"] + m["rot_dim"], None
+        mixer = {"heads": heads, "kv_heads": kv_heads, "dim": d, "vdim": d, "scale": d ** -0.5, "rot": {"base": 10000.0, "dims": d}}
+        if mask is not None:
+            mixer["mask"] = mask
+        out = {"type": "attention", "mixer": mixer, "mlp": {"kind": "dense", "ff": layer["mlp"]["ff"], "limit": layer["mlp"]["limit"]}}
+        if entry.layer in first:
+            out["weights_of"] = first[entry.layer]
+        else:
+            first[entry.layer] = i
+        layers.append(out)
+    return {"architecture": "Lanilix", "vocab": tur["vocab"], "width": tur["width"], "norm": tur["norm"], "layers": layers}
+
+
+def turutar_kernel_table(torch, tur, peak, batch, context):
+    """Every kernel of the Turutar design alone, beside the like kernel of the designs that have one: the
+    residual norms, windowed attention and products of Lanilix, the latent attention of Futepel."""
+    from thing_htn_2026_b200 import ops
+    from thing_htn_2026_b200.cache import KVSpec, SequenceCache
+    dev, bf = "cuda:0", torch.bfloat16
+    pick = lambda kind: next(l for l in tur["layers"] if l["type"] == kind)["mixer"]
+    win, lat = pick("attention"), pick("latent_attention")
+    W, T, V, ff = tur["width"], PREFILL_TOKENS, tur["vocab"], tur["layers"][0]["mlp"]["ff"]
+    side, table_width = tur["token_side"]["dim"], tur["token_side"]["dim"] * len(tur["layers"])
+    table = KernelTable(torch, peak)
+    row = table.row
+    g = torch.Generator(device=dev).manual_seed(0)
+    rnd = lambda *shape: torch.randn(shape, generator=g, device=dev)
+    err = ops.new_error_word(dev)
+    emb, side_table = rnd(V, W).to(bf), rnd(V, table_width).to(bf)
+    w_gate, w_proj = (rnd(side, W) * 0.02).to(bf), (rnd(W, side) * 0.1).to(bf)
+    around_zero, plain = ops.Gain(rnd(W) * 0.1, 1.0, 1e-6), ops.Gain(1 + rnd(W) * 0.1, 0.0, 1e-6)
+    s1, s2 = rnd(W), rnd(W)
+    H, G, D = win["heads"], win["kv_heads"], win["dim"]
+    width = (H + G) * D
+    padded = width + -(-H // 8) * 8
+    w_plain, w_in = (rnd(width, W) * 0.02).to(bf), (rnd(padded, W) * 0.02).to(bf)
+    b_in = rnd(padded).to(bf)
+    for m, tag in ((T, "prefill"), (batch, "decode")):
+        tokens = torch.randint(0, V, (m,), generator=g, device=dev, dtype=torch.int32)
+        h32, a16, f16, y16, start = rnd(m, W), rnd(m, W).to(bf), rnd(m, W).to(bf), rnd(m, W).to(bf), rnd(m, W)
+        row(f"{tag}: embed_norm (stream and its copy)", lambda: ops.embed_norm(emb, tokens, around_zero, err, copy=True),
+            nbytes=m * W * (2 + 8), like=f"{tag}: gather_rows_scaled")
+        row(f"{tag}: gather_rows_scaled", lambda: ops.gather_rows_scaled(emb, tokens, 8.0, err), nbytes=m * W * 6)
+        pair = ops.ScaledPair(a16, s1, f16, s2)
+        like = f"{tag}: residual_norm (norm of the branch, add, norm)"
+        row(f"{tag}: residual_norm (layer scale of two branches, the sum as it is)",
+            lambda: ops.residual_norm(h32, None, None, ops.STREAM_AS_IS, bf, scaled=pair), nbytes=m * W * (8 + 2 + 2 + 2), like=like)
+        row(f"{tag}: residual_norm (norm of the branch, add, the stream's start, norm)",
+            lambda: ops.residual_norm(h32, y16, plain, around_zero, bf, add_rows=start), nbytes=m * W * (8 + 2 + 4 + 2), like=like)
+        row(like, lambda: ops.residual_norm(h32, y16, around_zero, around_zero, bf), nbytes=m * W * (8 + 2 + 2))
+        row(f"{tag}: token_gate (product, gelu, the token's row)",
+            lambda: ops.token_gate(a16, w_gate, side_table, tokens, side, err), flops=2.0 * m * W * side,
+            nbytes=(m + side) * W * 2 + m * side * 4, like=f"{tag}: linear (of the gate's size), clamped_glu")
+        z = rnd(m, 2 * side).to(bf)
+        row(f"{tag}: linear (of the gate's size), clamped_glu",
+            lambda: (ops.linear(a16, w_gate, err=err), ops.clamped_glu(z, 7.0, 1.702)), flops=2.0 * m * W * side,
+            nbytes=(m + side) * W * 2 + m * side * 6)
+        z1 = rnd(m, side).to(bf)
+        row(f"{tag}: linear (the token part, back)", lambda: ops.linear(z1, w_proj, err=err), flops=2.0 * m * W * side,
+            nbytes=(m + W) * side * 2 + m * W * 2)
+        row(f"{tag}: linear (queries, keys and gates, biased)", lambda: ops.linear(a16, w_in, err=err, bias=b_in),
+            flops=2.0 * m * W * width, nbytes=(m + width) * W * 2 + m * width * 2, like=f"{tag}: linear (queries and keys)")
+        row(f"{tag}: linear (queries and keys)", lambda: ops.linear(a16, w_plain, err=err), flops=2.0 * m * W * width,
+            nbytes=(m + width) * W * 2 + m * width * 2)
+        proj, o16 = rnd(m, padded).to(bf), rnd(m, H * D).to(bf)
+        row(f"{tag}: logistic_gate (per head)", lambda: ops.logistic_gate(o16, proj, width, D), nbytes=m * H * (D * 4 + 2),
+            like=f"{tag}: logistic_gate")
+        row(f"{tag}: logistic_gate", lambda: ops.logistic_gate(o16, proj, 0), nbytes=m * H * D * 6)
+        gu = rnd(m, 2 * ff).to(bf)
+        row(f"{tag}: clamped_glu", lambda: ops.clamped_glu(gu, 7.0, 1.702), nbytes=m * ff * 6)
+
+    def over_a_cache(spec, prepare, widths, heads, scale, window, sinks, names, likes, cost_per_row, exact):
+        """Preparation and attention of a prompt, then of a decode step over ``context`` keys."""
+        cache = SequenceCache([spec], max_tokens=(batch * (context + 64) + T + 64), dtype=bf, device=dev, max_slots=batch + 2)
+        own = cache.open(batch + 1)
+        d, dv = spec.head_dim, spec.value_dim or spec.head_dim
+
+        def step_of(slot_list, counts):
+            cache.prepare(slot_list, counts)
+            cu = [0]
+            for c in counts:
+                cu.append(cu[-1] + c)
+            cu_dev, slots_dev = torch.tensor(cu, dtype=torch.int32, device=dev), torch.tensor(slot_list, dtype=torch.int32, device=dev)
+            return ops.step_rows(cu_dev, slots_dev, cache.seq_lens, cu[-1], max(counts),
+                                 max_context=max(cache.length(s) + c for s, c in zip(slot_list, counts)), lengths_differ=False), cu_dev, slots_dev
+
+        for n, who, tag in ((T, own[:1], "prefill"), (1, own[1:], "decode")):
+            if tag == "decode":
+                rows_, cu_dev, slots_dev = step_of(who, [context] * batch)
+                prepare([rnd(batch * context, w).to(bf) for w in widths], rows_, cache.kv_view(0))
+                ops.advance(cache.seq_lens, slots_dev, cu_dev)
+                cache.commit(who, [context] * batch)
+            rows_, cu_dev, slots_dev = step_of(who, [n] * len(who))
+            m = n * len(who)
+            inputs = [rnd(m, w).to(bf) for w in widths]
+            row(f"{tag}: {names[0]}", lambda: prepare(inputs, rows_, cache.kv_view(0)), nbytes=m * cost_per_row,
+                like=likes[0] and f"{tag}: {likes[0]}")
+            q = prepare(inputs, rows_, cache.kv_view(0))
+            tiles, size = None, ops.prompt_attention_tile(bf, d, 64, heads, spec.n_kv, dv) if n > 1 else 0
+            if size:
+                r0, rn = ops.row_tiles_of([n], [0], size)
+                tiles = ops.RowTiles(torch.tensor(r0, dtype=torch.int32, device=dev), torch.tensor(rn, dtype=torch.int32, device=dev),
+                                     len(r0), size)
+            seen = sum(min(i + 1, window or T) for i in range(T))
+            cost = dict(flops=2.0 * heads * (d + dv) * seen, nbytes=T * heads * (d + dv) * 2) if n > 1 else \
+                dict(nbytes=batch * spec.n_kv * min(context + 1, window or context + 1) * (d + dv) * 2)
+            row(f"{tag}: {names[1]}", lambda: ops.attention(q, rows_, cache.kv_view(0), heads, scale, window, err, tiles,
+                                                            exact_weights=exact, sinks=sinks),
+                like=likes[1] and f"{tag}: {likes[1]}", **cost)
+
+    # ---- windowed attention: this design's, then Lanilix's (rotated keys, no sink, no gate rows)
+    qg, kg, window = 1 + rnd(H * D) * 0.1, 1 + rnd(G * D) * 0.1, win["mask"]["size"]
+    turn = ops.RotaryTables(torch.ones(8192, D // 2, device=dev), torch.zeros(8192, D // 2, device=dev), D, "interleaved")
+    for rotary, row_width, sinks, names, likes, exact in (
+            (turn, width, None, ("qk_prepare (rotated)", f"attention (window {window})"), (None, None), False),
+            (None, padded, torch.zeros(H, device=dev), ("qk_prepare", f"attention (window {window}, one added)"),
+             ("qk_prepare (rotated)", f"attention (window {window})"), True)):
+        over_a_cache(KVSpec(G, D, window), lambda x, rows_, kv: ops.qk_prepare(x[0], qg, kg, "projection", 1e-6, rotary, rows_, kv, H,
+                                                                               True, True, err),
+                     [row_width], H, win["scale"], window, sinks, names, likes, (width + (H + 2 * G) * D) * 2, exact)
+
+    # ---- latent attention: this design's, then Futepel's (queries by one product, no sinks)
+    Hl, P, R, E, C, Q = lat["heads"], lat["dim"], lat["rot_dim"], lat["vdim"], lat["kv_rank"], lat["q_rank"]
+    D = P + R
+    turn_l = ops.RotaryTables(torch.ones(8192, R // 2, device=dev), torch.zeros(8192, R // 2, device=dev), R, "interleaved")
+    gain_c, gain_q = 1 + rnd(C) * 0.1, 1 + rnd(Q) * 0.1
+
+    def plain_queries(x, rows_, kv):
+        ops.latent_norm(x[0], Hl * D, C, gain_c, 1e-6)
+        return ops.latent_assemble(x[0], 0, Hl * D + C, x[1], turn_l, rows_, kv, Hl, P, R, err)
+
+    def latent_queries(x, rows_, kv):
+        ops.latent_norm(x[0], 0, Q, gain_q, 1e-6, second=(Q, C, gain_c))
+        return ops.latent_assemble(x[0], 0, Q + C, x[1], turn_l, rows_, kv, Hl, P, R, err, q_rows=x[2])
+
+    common = Hl * (P + E) * 2 + (2 * C + R) * 2 + Hl * D * 4 + Hl * (D + E) * 2
+    over_a_cache(KVSpec(Hl, D, None, 0, None, E), plain_queries, [Hl * D + C + R + Hl, Hl * (P + E)], Hl, lat["scale"], None, None,
+                 ("latent_norm + latent_assemble", "attention (latent heads)"), (None, None), common, True)
+    over_a_cache(KVSpec(Hl, D, None, 0, None, E), latent_queries, [Q + C + R + Hl, Hl * (P + E), Hl * D], Hl, lat["scale"], None, rnd(Hl),
+                 ("latent_norm (two) + latent_assemble", "attention (latent heads, sinks)"),
+                 ("latent_norm + latent_assemble", "attention (latent heads)"), common + Q * 4, True)
+    for m, tag in ((T, "prefill"), (batch, "decode")):
+        n16, cq, c16 = rnd(m, W).to(bf), rnd(m, Q).to(bf), rnd(m, C).to(bf)
+        w_dq, w_uq, w_q = (rnd(Q, W) * 0.02).to(bf), (rnd(Hl * D, Q) * 0.02).to(bf), (rnd(Hl * D, W) * 0.02).to(bf)
+        row(f"{tag}: linear (queries out of their latent)", lambda: ops.linear(cq, w_uq, err=err), flops=2.0 * m * Q * Hl * D,
+            nbytes=(m + Hl * D) * Q * 2 + m * Hl * D * 2, like=f"{tag}: linear (latent heads' queries, one product)")
+        row(f"{tag}: linear (latent heads' queries, one product)", lambda: ops.linear(n16, w_q, err=err), flops=2.0 * m * W * Hl * D,
+            nbytes=(m + Hl * D) * W * 2 + m * Hl * D * 2)
+    ops.raise_on_device_error(err, "kernel table")
+    return table.finished()
+
+
 def run_design(args):
     import torch
     from thing_htn_2026_b200 import Engine, ops
@@ -1549,7 +1721,7 @@ def run_design(args):
     ops.launch_count = 0
     design = args.design
     design_sizes = {"lanilix": DESIGN_SIZES, "bunudra": BUNUDRA_SIZES, "ditilix": DITILIX_SIZES, "dubazen": DUBAZEN_SIZES,
-                    "futepel": FUTEPEL_SIZES}[design]
+                    "futepel": FUTEPEL_SIZES, "turutar": TURUTAR_SIZES}[design]
     for name in design_sizes:
         lan = named_config_json(name)
         if args.layers:
@@ -1561,7 +1733,8 @@ def run_design(args):
                   "bunudra": lambda: ("lanilix_same_size", lanilix_like(lan)),
                   "ditilix": lambda: ("qwen3_same_size", qwen3_like_ditilix(lan)),
                   "dubazen": lambda: ("bunudra_same_size", bunudra_like(lan)),
-                  "futepel": lambda: ("bunudra_same_size", bunudra_like_futepel(lan))}[design]()
+                  "futepel": lambda: ("bunudra_same_size", bunudra_like_futepel(lan)),
+                  "turutar": lambda: ("lanilix_same_size", lanilix_like_turutar(lan))}[design]()
         for label, data in ((design, lan), beside):
             engine = Engine.from_config(config_from_dict(data), seed=0, dtype="bfloat16", max_tokens=max_tokens,
                                         max_batch=args.batch)
@@ -1570,7 +1743,8 @@ def run_design(args):
             del engine
             torch.cuda.empty_cache()
         table = {"lanilix": kernel_table, "bunudra": bunudra_kernel_table, "ditilix": ditilix_kernel_table,
-                 "dubazen": dubazen_kernel_table, "futepel": futepel_kernel_table}[design]
+                 "dubazen": dubazen_kernel_table, "futepel": futepel_kernel_table,
+                 "turutar": turutar_kernel_table}[design]
         entry["kernels"] = table(torch, lan, peak, args.batch, args.prompt_len)
         sizes[name] = entry
     clocks = sampler.stop()
@@ -1785,9 +1959,9 @@ def main():
                              "(for ncu --profile-from-start off)")
     parser.add_argument("--workload", choices=sorted(LARGE_WORKLOADS), default=None,
                         help="one of the two larger workloads instead of the default run")
-    parser.add_argument("--design", choices=["lanilix", "bunudra", "ditilix", "dubazen", "futepel"], default=None,
+    parser.add_argument("--design", choices=["lanilix", "bunudra", "ditilix", "dubazen", "futepel", "turutar"], default=None,
                         help="another design beside its closest relative at the same sizes (Lanilix beside Qwen3, "
-                             "Bunudra beside Lanilix, Ditilix beside Qwen3, Dubazen and Futepel beside Bunudra), model by model and kernel by kernel, "
+                             "Bunudra beside Lanilix, Ditilix beside Qwen3, Dubazen and Futepel beside Bunudra, Turutar beside Lanilix), model by model and kernel by kernel, "
                              "instead of the default run")
     args = parser.parse_args()
     args.steps_given = args.steps is not None
