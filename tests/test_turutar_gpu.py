@@ -255,6 +255,30 @@ def test_the_gate_of_the_token_part(dtype, rows, width, dim, column, table_width
         err.zero_()
 
 
+@pytest.mark.parametrize("rows, width, dim, second", [(1, 48, 10, True), (8, 2048, 128, True), (16, 72, 16, False), (5, 4096, 256, True),
+                                                      (3, 8, 3, True), (2, 16384, 5, True)])
+def test_the_gate_of_the_token_part_behind_pending_outputs(rows, width, dim, second):
+    """The kernel that adds up the stream and what is pending on it for itself: the same bits as adding
+    first, and the stream stays as it is."""
+    from thing_htn_2026_b200 import ops
+    bf = torch.bfloat16
+    h, a, f = rand((rows, width), 1).to(DEV), rand((rows, width), 2).to(bf).to(DEV), rand((rows, width), 3).to(bf).to(DEV)
+    s1, s2 = rand((width,), 4).to(DEV), rand((width,), 5).to(DEV)
+    w, table = rand((dim, width), 6, 2.0 / math.sqrt(width)).to(bf).to(DEV), rand((20, 2 * dim), 7).to(bf).to(DEV)
+    toks = torch.arange(rows, dtype=torch.int32, device=DEV) + 2
+    err = ops.new_error_word(DEV)
+    pair = ops.ScaledPair(a, s1, f if second else None, s2 if second else None)
+    before = h.clone()
+    got = ops.token_gate_pending(h, pair, w, table, toks, dim, err)
+    assert torch.equal(h, before)
+    _, x = ops.residual_norm(h, None, None, ops.STREAM_AS_IS, bf, scaled=pair)
+    assert torch.equal(got, ops.token_gate(x, w, table, toks, dim, err, fused=True))
+    z = x.cpu().double() @ w.cpu().double().t()
+    want = torch.nn.functional.gelu(z, approximate="tanh") * table.cpu().double()[2:2 + rows, dim:]
+    close(got, want, "bfloat16", "token gate behind pending outputs", 0.3)
+    assert int(err.item()) == 0
+
+
 @pytest.mark.parametrize("dtype", DTYPES)
 @pytest.mark.parametrize("name", [n for n in tiny.CONFIGS if tiny.CONFIGS[n]["side"]])
 def test_the_token_part_alone(models, dtype, name):
@@ -307,6 +331,81 @@ def test_feed_forward_alone(models, dtype, name, layer):
     up, gate = x.float() @ w[prefix + "up"].t(), x.float() @ w[prefix + "gate"].t()
     assert (up > mlp["limit"]).any() and (up < -mlp["limit"]).any() and (gate > mlp["limit"]).any()
     close(part.forward(x.to(DEV), None), plain.clamped_feed_forward(ar, x.float(), w, prefix, mlp["limit"]), dtype, "feed-forward")
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("inter, offset, more", [(40, 16, 0), (56, 8, 24), (7, 3, 2), (4096, 2568, 0)])
+def test_gates_and_ups_out_of_wider_rows(dtype, inter, offset, more):
+    from thing_htn_2026_b200 import ops
+    t = TORCH[dtype]
+    proj = rand((9, offset + 2 * inter + more), 1, 2.0).to(t)
+    g, u = (proj.double()[:, offset + k * inter:offset + (k + 1) * inter] for k in (0, 1))
+    g, u = g.clamp(max=1.5), u.clamp(-1.5, 1.5)
+    close(ops.clamped_glu(proj.to(DEV), 1.5, 1.702, offset, inter), g * torch.sigmoid(1.702 * g) * (u + 1.0), dtype, "slice", 0.3)
+    with pytest.raises(ops.KernelError, match="hold no"):
+        ops.clamped_glu(proj.to(DEV), 1.5, 1.702, offset + more + 1, inter)
+
+
+def test_work_beside_the_current_stream():
+    """What a second stream computes from what came before it, read after the join, again and again over the
+    same memory; counters of its own; not nested; the same in a captured graph."""
+    from thing_htn_2026_b200 import ops
+    beside = ops.Beside(DEV)
+    x, w1, w2 = rand((8, 4096), 1).to(torch.bfloat16).to(DEV), rand((256, 4096), 2, 0.02).to(torch.bfloat16).to(DEV), rand((384, 4096), 3, 0.02).to(torch.bfloat16).to(DEV)
+    err = ops.new_error_word(DEV)
+
+    def both(x):
+        y = ops.linear_stream(x, w1, err=err)
+        for _ in range(3):
+            z = ops.squared_relu(x)
+            with beside:
+                f = ops.linear_stream(z, w2, err=err)
+                with pytest.raises(ops.KernelError, match="nested"):
+                    with beside:
+                        pass
+            y = y + ops.linear_stream(z, w1, err=err)
+            beside.join()
+            y = y + f[:, :256]
+        return y
+
+    with torch.inference_mode():
+        z = ops.squared_relu(x)
+        want = ops.linear_stream(x, w1)
+        for _ in range(3):
+            want = want + ops.linear_stream(z, w1) + 0.0
+            want = want + ops.linear_stream(z, w2)[:, :256]
+        for _ in range(5):
+            assert torch.equal(both(x), want)
+        graph = torch.cuda.CUDAGraph()
+        with torch.cuda.graph(graph):
+            out = both(x)
+        for _ in range(5):
+            graph.replay()
+        torch.cuda.synchronize()
+        assert torch.equal(out, want) and int(err.item()) == 0
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("name", ["a", "c", "d"])
+def test_one_product_for_both_sublayers(models, dtype, name):
+    """A layer whose sublayers share their input product holds every weight once and gives what the
+    sublayers give with products of their own, alone and on two streams."""
+    from thing_htn_2026_b200.config import load_config
+    from thing_htn_2026_b200.engine.loading import load_model
+    model = load_model(models[name], dtype, DEV)
+    for i, layer in enumerate(load_config(models[name]).to_dict()["layers"]):
+        block = model.layers[i]
+        if layer["mlp"] is None:
+            assert block.w_in is None and block.ffn is None
+            continue
+        assert block.w_in.shape[0] % 8 == 0 and block.ffn_offset % 8 == 0
+        assert block.ffn.w_gate_up.data_ptr() == block.w_in[block.ffn_offset:].data_ptr()
+        own = block.mixer.w_qkv if layer["type"] == "attention" else block.mixer.w_in
+        assert own.data_ptr() == block.w_in.data_ptr()
+        x = rand((5, block.w_in.shape[1]), i).to(TORCH[dtype]).to(DEV)
+        from thing_htn_2026_b200 import ops
+        proj = ops.linear(x, block.w_in, bias=block.b_in)
+        close(block.ffn.forward_rows(proj, block.ffn_offset, None), block.ffn.forward(x, None), dtype, f"layer {i}", 0.3)
 
 
 # ----------------------------------------------------------------------------- mixers alone

@@ -748,31 +748,31 @@ THN_API int thn_swiglu(void* out, const void* gu, int rows, int inter, int dtype
 // out[m, i] = g s(alpha g) (u + 1) with g = min(gu[m, i], limit), u = clamp(gu[m, inter + i], -limit, limit)
 // and s the logistic function; float32 inside, rounded once.
 template <typename T>
-__global__ void clamped_glu_kernel(T* __restrict__ out, const T* __restrict__ gu, long long total, int inter, float limit,
-                                   float alpha) {
+__global__ void clamped_glu_kernel(T* __restrict__ out, const T* __restrict__ gu, long long row_stride, long long total,
+                                   int inter, float limit, float alpha) {
     pdl_launch_dependents();
     pdl_wait();
     const long long stride = (long long)gridDim.x * blockDim.x;
     for (long long e = (long long)blockIdx.x * blockDim.x + threadIdx.x; e < total; e += stride) {
         const long long m = e / inter;
         const int i = (int)(e - m * inter);
-        const float g = fminf(to_f32<T>(gu[m * 2 * inter + i]), limit);
-        const float u = fminf(fmaxf(to_f32<T>(gu[m * 2 * inter + inter + i]), -limit), limit);
+        const float g = fminf(to_f32<T>(gu[m * row_stride + i]), limit);
+        const float u = fminf(fmaxf(to_f32<T>(gu[m * row_stride + inter + i]), -limit), limit);
         out[e] = from_f32<T>(g / (1.0f + expf(-alpha * g)) * (u + 1.0f));
     }
 }
 
 // bfloat16 with inter % 8 == 0: eight values per thread, 16-byte accesses, the same arithmetic.
 __global__ void clamped_glu_bf16_vec_kernel(__nv_bfloat16* __restrict__ out, const __nv_bfloat16* __restrict__ gu,
-                                            long long total_vecs, int inter_vecs, float limit, float alpha) {
+                                            long long row_vecs, long long total_vecs, int inter_vecs, float limit, float alpha) {
     pdl_launch_dependents();
     pdl_wait();
     const long long stride = (long long)gridDim.x * blockDim.x;
     for (long long e = (long long)blockIdx.x * blockDim.x + threadIdx.x; e < total_vecs; e += stride) {
         const long long m = e / inter_vecs;
         const int i = (int)(e - m * inter_vecs);
-        const uint4 gv = *reinterpret_cast<const uint4*>(gu + (m * 2 * inter_vecs + i) * 8);
-        const uint4 uv = *reinterpret_cast<const uint4*>(gu + (m * 2 * inter_vecs + inter_vecs + i) * 8);
+        const uint4 gv = *reinterpret_cast<const uint4*>(gu + (m * row_vecs + i) * 8);
+        const uint4 uv = *reinterpret_cast<const uint4*>(gu + (m * row_vecs + inter_vecs + i) * 8);
         const __nv_bfloat162* g2 = reinterpret_cast<const __nv_bfloat162*>(&gv);
         const __nv_bfloat162* u2 = reinterpret_cast<const __nv_bfloat162*>(&uv);
         uint4 ov;
@@ -789,29 +789,30 @@ __global__ void clamped_glu_bf16_vec_kernel(__nv_bfloat16* __restrict__ out, con
     }
 }
 
-// gu [rows, 2 * inter] (gate columns, then up columns) -> out [rows, inter].
-THN_API int thn_clamped_glu(void* out, const void* gu, int rows, int inter, float limit, float alpha, int dtype,
+// gu: rows of 2 * inter (gate columns, then up columns), row_stride elements apart -> out [rows, inter].
+THN_API int thn_clamped_glu(void* out, const void* gu, long long row_stride, int rows, int inter, float limit, float alpha, int dtype,
                             cudaStream_t stream) {
     THN_CHECK_ARG(rows >= 0 && inter > 0 && limit > 0.f, "clamped_glu: bad sizes rows=%d inter=%d limit=%g", rows, inter,
                   (double)limit);
+    THN_CHECK_ARG(row_stride >= 2LL * inter, "clamped_glu: rows %lld apart are too short for %d gates and ups", row_stride, inter);
     const long long total = (long long)rows * inter;
     if (total == 0) return THN_OK;
     const int threads = 256;
     const long long want = (total + threads - 1) / threads;
     const int blocks = (int)(want < 148 * 16 ? want : 148 * 16);
-    if (dtype == THN_BF16 && inter % 8 == 0 && (((uintptr_t)gu | (uintptr_t)out) & 15) == 0) {
+    if (dtype == THN_BF16 && inter % 8 == 0 && row_stride % 8 == 0 && (((uintptr_t)gu | (uintptr_t)out) & 15) == 0) {
         const long long vecs = total / 8;
         const long long want_vec = (vecs + threads - 1) / threads;
         thn_launch(clamped_glu_bf16_vec_kernel, (unsigned)(want_vec < 148 * 32 ? want_vec : 148 * 32), threads, 0, stream,
-                   (__nv_bfloat16*)out, (const __nv_bfloat16*)gu, vecs, inter / 8, limit, alpha);
+                   (__nv_bfloat16*)out, (const __nv_bfloat16*)gu, row_stride / 8, vecs, inter / 8, limit, alpha);
         return thn_launch_status("clamped_glu");
     }
     if (dtype == THN_F32)
-        thn_launch(clamped_glu_kernel<float>, blocks, threads, 0, stream, (float*)out, (const float*)gu, total, inter,
+        thn_launch(clamped_glu_kernel<float>, blocks, threads, 0, stream, (float*)out, (const float*)gu, row_stride, total, inter,
                    limit, alpha);
     else if (dtype == THN_BF16)
         thn_launch(clamped_glu_kernel<__nv_bfloat16>, blocks, threads, 0, stream, (__nv_bfloat16*)out,
-                   (const __nv_bfloat16*)gu, total, inter, limit, alpha);
+                   (const __nv_bfloat16*)gu, row_stride, total, inter, limit, alpha);
     else
         THN_CHECK_ARG(false, "clamped_glu: unknown dtype %d", dtype);
     return thn_launch_status("clamped_glu");

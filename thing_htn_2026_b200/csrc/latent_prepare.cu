@@ -46,6 +46,45 @@ __global__ void __launch_bounds__(128) latent_norm_kernel(Latent one, Latent two
     for (int i = threadIdx.x; i < l.rank; i += blockDim.x) out[i] = from_f32<T>(to_f32<T>(row[i]) * r * l.gain[i]);
 }
 
+// The same for bfloat16 in 16-byte pieces; a thread's first piece stays in registers between the two passes.
+__global__ void __launch_bounds__(128) latent_norm_vec_kernel(Latent one, Latent two, const __nv_bfloat16* __restrict__ src,
+                                                              long long src_stride, float eps) {
+    pdl_launch_dependents();
+    pdl_wait();
+    __shared__ float scratch[33];
+    const Latent l = blockIdx.y ? two : one;
+    const uint4* row = reinterpret_cast<const uint4*>(src + (size_t)blockIdx.x * src_stride + l.offset);
+    uint4* out = reinterpret_cast<uint4*>((__nv_bfloat16*)l.out + (size_t)blockIdx.x * l.rank);
+    const int pieces = l.rank / 8;
+    uint4 first = make_uint4(0, 0, 0, 0);
+    float ss = 0.f;
+    for (int i = threadIdx.x; i < pieces; i += 128) {
+        const uint4 raw = row[i];
+        if (i < 128) first = raw;
+        const __nv_bfloat162* x = reinterpret_cast<const __nv_bfloat162*>(&raw);
+#pragma unroll
+        for (int j = 0; j < 4; ++j) {
+            const float2 v = __bfloat1622float2(x[j]);
+            ss += v.x * v.x + v.y * v.y;
+        }
+    }
+    const float r = 1.0f / sqrtf(block_sum(ss, scratch) / (float)l.rank + eps);
+    for (int i = threadIdx.x; i < pieces; i += 128) {
+        const uint4 raw = i < 128 ? first : row[i];
+        const float4 g0 = reinterpret_cast<const float4*>(l.gain)[2 * i], g1 = reinterpret_cast<const float4*>(l.gain)[2 * i + 1];
+        const float g[8] = {g0.x, g0.y, g0.z, g0.w, g1.x, g1.y, g1.z, g1.w};
+        const __nv_bfloat162* x = reinterpret_cast<const __nv_bfloat162*>(&raw);
+        uint4 packed;
+        __nv_bfloat162* o = reinterpret_cast<__nv_bfloat162*>(&packed);
+#pragma unroll
+        for (int j = 0; j < 4; ++j) {
+            const float2 v = __bfloat1622float2(x[j]);
+            o[j] = __floats2bfloat162_rn(v.x * r * g[2 * j], v.y * r * g[2 * j + 1]);
+        }
+        out[i] = packed;
+    }
+}
+
 template <typename T>
 __global__ void __launch_bounds__(256) latent_assemble_kernel(
     T* __restrict__ q_out, const T* __restrict__ q_src, long long q_stride, const T* __restrict__ shared_src,
@@ -214,7 +253,11 @@ THN_API int thn_latent_norm(void* out, long long offset, const float* gain, int 
     if (rows == 0) return THN_OK;
     const Latent one{out, gain, offset, rank}, two{out2, gain2, offset2, rank2};
     const dim3 grid(rows, out2 ? 2 : 1);
-    if (dtype == THN_F32)
+    const bool whole = ((rank | (out2 ? rank2 : 0) | (int)(src_stride % 8) | (int)(offset % 8) | (int)(out2 ? offset2 % 8 : 0)) % 8) == 0 &&
+                       (((uintptr_t)out | (uintptr_t)out2 | (uintptr_t)src | (uintptr_t)gain | (uintptr_t)gain2) & 15) == 0;
+    if (dtype == THN_BF16 && whole)
+        thn_launch(latent_norm_vec_kernel, grid, 128, 0, stream, one, two, (const __nv_bfloat16*)src, src_stride, eps);
+    else if (dtype == THN_F32)
         thn_launch(latent_norm_kernel<float>, grid, 128, 0, stream, one, two, (const float*)src, src_stride, eps);
     else if (dtype == THN_BF16)
         thn_launch(latent_norm_kernel<__nv_bfloat16>, grid, 128, 0, stream, one, two, (const __nv_bfloat16*)src, src_stride, eps);

@@ -7,7 +7,9 @@
 // token_gate takes z as the product gave it.  token_gate_product computes z = W x as well, for steps of few
 // rows: a block of eight warps takes one row and walks the outputs four at a time (16-byte pieces of the row
 // and of four weight rows side by side, float32 sums over the warp by shuffles and over the warps in a fixed
-// order), so that a row's result depends on nothing but the sizes.
+// order), so that a row's result depends on nothing but the sizes.  With a pending pair of branch outputs the
+// row is h + (s p + s' p'), rounded to the activation type: the block adds it up for itself and leaves h as
+// it is (several blocks read it); whoever adds the token part to the stream adds the pair as well.
 // A token outside the table sets THN_ERR_TOKEN_RANGE and reads row 0.
 #include "common.cuh"
 
@@ -79,15 +81,66 @@ __device__ __forceinline__ float dot8(const uint4& a, const uint4& b, float acc)
 
 constexpr int kProductThreads = 256;
 
+// The stream and the outputs that are still to be added to it (second may be null).
+struct Pending {
+    const float* h;
+    const __nv_bfloat16 *first, *second;
+    const float *scale1, *scale2;
+};
+
+__device__ __forceinline__ void eight(const float* p, float (&v)[8]) {
+    const float4 a = reinterpret_cast<const float4*>(p)[0], b = reinterpret_cast<const float4*>(p)[1];
+    v[0] = a.x, v[1] = a.y, v[2] = a.z, v[3] = a.w, v[4] = b.x, v[5] = b.y, v[6] = b.z, v[7] = b.w;
+}
+__device__ __forceinline__ void eight(const __nv_bfloat16* p, float (&v)[8]) {
+    const uint4 raw = *reinterpret_cast<const uint4*>(p);
+    const __nv_bfloat162* pairs = reinterpret_cast<const __nv_bfloat162*>(&raw);
+#pragma unroll
+    for (int k = 0; k < 4; ++k) {
+        const float2 f = __bfloat1622float2(pairs[k]);
+        v[2 * k] = f.x, v[2 * k + 1] = f.y;
+    }
+}
+
+template <bool PENDING>
 __global__ void __launch_bounds__(kProductThreads) token_gate_product_kernel(
-    __nv_bfloat16* __restrict__ out, const __nv_bfloat16* __restrict__ x, const __nv_bfloat16* __restrict__ w,
+    __nv_bfloat16* __restrict__ out, const __nv_bfloat16* __restrict__ x, Pending pending, const __nv_bfloat16* __restrict__ w,
     const __nv_bfloat16* __restrict__ table, const int* __restrict__ tokens, int dim, int vecs, long long table_width,
     int column0, int n_table_rows, int* __restrict__ err) {
     pdl_launch_dependents();
+    // the weight's rows of this block, into L2 while the kernel before still runs
+    for (int n0 = blockIdx.y * 4; n0 < dim; n0 += gridDim.y * 4)
+        for (int j = 0; j < 4 && n0 + j < dim; ++j)
+            for (int i = threadIdx.x * 8; i < vecs; i += kProductThreads * 8)
+                asm volatile("prefetch.global.L2 [%0];" ::"l"(reinterpret_cast<const uint4*>(w) + (size_t)(n0 + j) * vecs + i));
     pdl_wait();
+    extern __shared__ uint4 row[];          // PENDING: the row, rounded
     __shared__ float part[kProductThreads / 32][4];
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, m = blockIdx.x;
-    const uint4* a = reinterpret_cast<const uint4*>(x) + (size_t)m * vecs;
+    const uint4* a = PENDING ? row : reinterpret_cast<const uint4*>(x) + (size_t)m * vecs;
+    if (PENDING) {
+        const size_t base = (size_t)m * vecs * 8;
+        for (int i = threadIdx.x; i < vecs; i += kProductThreads) {     // a thread reads back only what it wrote
+            float v[8], s[8], p[8], f[8];
+            eight(pending.h + base + i * 8, v);
+            eight(pending.first + base + i * 8, s);
+            eight(pending.scale1 + i * 8, f);
+#pragma unroll
+            for (int e = 0; e < 8; ++e) s[e] *= f[e];
+            if (pending.second) {
+                eight(pending.second + base + i * 8, p);
+                eight(pending.scale2 + i * 8, f);
+#pragma unroll
+                for (int e = 0; e < 8; ++e) s[e] = fmaf(p[e], f[e], s[e]);
+            }
+            uint4 packed;
+            __nv_bfloat162* o2 = reinterpret_cast<__nv_bfloat162*>(&packed);
+#pragma unroll
+            for (int k = 0; k < 4; ++k)
+                o2[k] = __floats2bfloat162_rn(__fadd_rn(v[2 * k], s[2 * k]), __fadd_rn(v[2 * k + 1], s[2 * k + 1]));
+            row[i] = packed;
+        }
+    }
     const uint4* wv = reinterpret_cast<const uint4*>(w);
     const uint4 zero = make_uint4(0, 0, 0, 0);
     for (int n0 = blockIdx.y * 4; n0 < dim; n0 += gridDim.y * 4) {
@@ -143,18 +196,33 @@ THN_API int thn_token_gate(void* out, const void* z, const void* table, const in
     return thn_launch_status("token_gate");
 }
 
-// x [rows, width] and w [dim, width] bfloat16, 16-byte aligned, width a multiple of eight.
-THN_API int thn_token_gate_product_bf16(void* out, const void* x, const void* w, const void* table, const int* tokens, int rows,
-                                        int width, int dim, int table_width, int column0, int n_table_rows, int* err,
-                                        cudaStream_t stream) {
+// x [rows, width] and w [dim, width] bfloat16, 16-byte aligned, width a multiple of eight.  With h (float32
+// [rows, width]) instead of x: the row is h + scale1 first + scale2 second (second and scale2 may be null).
+THN_API int thn_token_gate_product_bf16(void* out, const void* x, const float* h, const void* first, const float* scale1,
+                                        const void* second, const float* scale2, const void* w, const void* table,
+                                        const int* tokens, int rows, int width, int dim, int table_width, int column0,
+                                        int n_table_rows, int* err, cudaStream_t stream) {
     THN_CHECK_ARG(rows >= 0 && dim > 0 && width > 0 && width % 8 == 0 && column0 >= 0 && column0 + dim <= table_width &&
                       n_table_rows > 0,
                   "token_gate_product: bad sizes rows=%d width=%d dim=%d", rows, width, dim);
-    THN_CHECK_ARG((((uintptr_t)x | (uintptr_t)w) & 15) == 0, "token_gate_product: operands must be 16-byte aligned (rows=%d)", rows);
+    THN_CHECK_ARG((x == nullptr) != (h == nullptr), "token_gate_product: a row, or a stream with what is pending (rows=%d)", rows);
+    THN_CHECK_ARG(h == nullptr || (first && scale1 && (second == nullptr) == (scale2 == nullptr)),
+                  "token_gate_product: pending outputs come with their factors (rows=%d)", rows);
+    THN_CHECK_ARG((((uintptr_t)x | (uintptr_t)w | (uintptr_t)h | (uintptr_t)first | (uintptr_t)scale1 | (uintptr_t)second |
+                    (uintptr_t)scale2) & 15) == 0, "token_gate_product: operands must be 16-byte aligned (rows=%d)", rows);
     if (rows == 0) return THN_OK;
     const int groups = (dim + 3) / 4, want = (2 * 148 + rows - 1) / rows;
-    thn_launch(token_gate_product_kernel, dim3(rows, groups < want ? groups : want), kProductThreads, 0, stream,
-               (__nv_bfloat16*)out, (const __nv_bfloat16*)x, (const __nv_bfloat16*)w, (const __nv_bfloat16*)table, tokens, dim,
-               width / 8, (long long)table_width, column0, n_table_rows, err);
+    const dim3 grid(rows, groups < want ? groups : want);
+    const Pending pending{h, (const __nv_bfloat16*)first, (const __nv_bfloat16*)second, scale1, scale2};
+    const size_t smem = h ? (size_t)width * 2 : 0;
+    THN_UNSUPPORTED_IF(smem > 40 * 1024, "token_gate_product: rows of %d values do not fit shared memory", width);
+    if (h)
+        thn_launch(token_gate_product_kernel<true>, grid, kProductThreads, smem, stream, (__nv_bfloat16*)out,
+                   (const __nv_bfloat16*)x, pending, (const __nv_bfloat16*)w, (const __nv_bfloat16*)table, tokens, dim, width / 8,
+                   (long long)table_width, column0, n_table_rows, err);
+    else
+        thn_launch(token_gate_product_kernel<false>, grid, kProductThreads, smem, stream, (__nv_bfloat16*)out,
+                   (const __nv_bfloat16*)x, pending, (const __nv_bfloat16*)w, (const __nv_bfloat16*)table, tokens, dim, width / 8,
+                   (long long)table_width, column0, n_table_rows, err);
     return thn_launch_status("token_gate_product");
 }

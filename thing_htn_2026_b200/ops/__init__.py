@@ -63,8 +63,8 @@ _SIGNATURES = {
     "thn_embed_norm": [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_float, c_float, c_int, c_int, c_int, c_int,
                        c_void_p, c_void_p],
     "thn_token_gate": [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p],
-    "thn_token_gate_product_bf16": [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int,
-                                    c_void_p, c_void_p],
+    "thn_token_gate_product_bf16": [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
+                                    c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p],
     "thn_gated_head_norm": [c_void_p, c_void_p, c_void_p, c_longlong, c_void_p, c_float, c_int, c_int, c_int, c_int,
                             c_int, c_longlong, c_float, c_int, c_void_p],
     "thn_hyper_norm": [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_float,
@@ -117,7 +117,7 @@ _SIGNATURES = {
     "thn_moe_route": [c_void_p, c_void_p, c_void_p, c_void_p, c_longlong, c_int, c_int, c_int, c_int, c_int, c_float,
                       c_int, c_int, c_float, c_void_p],
     "thn_routed_gelu": [c_void_p, c_void_p, c_void_p, c_void_p, c_longlong, c_int, c_int, c_int, c_int, c_int, c_void_p],
-    "thn_clamped_glu": [c_void_p, c_void_p, c_int, c_int, c_float, c_float, c_int, c_void_p],
+    "thn_clamped_glu": [c_void_p, c_void_p, c_longlong, c_int, c_int, c_float, c_float, c_int, c_void_p],
     "thn_qk_prepare": [c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_int, c_float, c_float, c_void_p, c_void_p,
                        c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int,
                        c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p, c_void_p],
@@ -496,16 +496,21 @@ def swiglu(gu: torch.Tensor) -> torch.Tensor:
     return out
 
 
-def clamped_glu(gu: torch.Tensor, limit: float, alpha: float) -> torch.Tensor:
+def clamped_glu(gu: torch.Tensor, limit: float, alpha: float, offset: int = 0, inter: Optional[int] = None) -> torch.Tensor:
     """gu [rows, 2*I] (gate columns first) -> g * logistic(alpha * g) * (u + 1) with
-    g = min(gate, limit) and u = clamp(up, -limit, limit), [rows, I]."""
+    g = min(gate, limit) and u = clamp(up, -limit, limit), [rows, I].  With ``inter`` (I) the gates and ups are
+    the 2*I columns from ``offset`` of wider rows."""
     _need(gu, "clamped_glu")
     rows, width = gu.shape
-    if width % 2:
-        raise KernelError(f"clamped_glu: width {width} is odd")
-    out = torch.empty((rows, width // 2), dtype=gu.dtype, device=gu.device)
-    _call("thn_clamped_glu", _ptr(out), _ptr(gu), rows, width // 2, float(limit), float(alpha), _code(gu, "clamped_glu"),
-          _stream())
+    if inter is None:
+        if width % 2 or offset:
+            raise KernelError(f"clamped_glu: width {width} is odd, or an offset without a size")
+        inter = width // 2
+    if offset < 0 or offset + 2 * inter > width:
+        raise KernelError(f"clamped_glu: rows of {width} hold no {inter} gates and ups from column {offset}")
+    out = torch.empty((rows, inter), dtype=gu.dtype, device=gu.device)
+    _call("thn_clamped_glu", _ptr(out), gu.data_ptr() + offset * gu.element_size(), width, rows, inter, float(limit),
+          float(alpha), _code(gu, "clamped_glu"), _stream())
     return out
 
 
@@ -607,6 +612,39 @@ def residual_norm(h: Optional[torch.Tensor], d: Optional[torch.Tensor], post: Op
     return h, y
 
 
+TOKEN_GATE_PENDING_WIDTH = 16384
+
+
+def token_gate_pending_supported(h: torch.Tensor, weight: torch.Tensor) -> bool:
+    width = weight.shape[1]
+    return weight.dtype == torch.bfloat16 and h.dtype == torch.float32 and width % 8 == 0 and width <= TOKEN_GATE_PENDING_WIDTH
+
+
+def token_gate_pending(h: torch.Tensor, scaled: ScaledPair, weight: torch.Tensor, table: torch.Tensor, tokens: torch.Tensor,
+                       column: int, err: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """:func:`token_gate` for few rows of bfloat16 activations, reading ``h + scaled`` (rounded) while the
+    outputs in ``scaled`` are still to be added to the float32 stream ``h``, which stays as it is."""
+    dim, width = weight.shape
+    _need(h, "token_gate_pending h", torch.float32)
+    _need(weight, "token_gate_pending weight", torch.bfloat16)
+    _need(table, "token_gate_pending table", torch.bfloat16)
+    _need(tokens, "token_gate_pending tokens", torch.int32)
+    for t, s in ((scaled.first, scaled.scale1), (scaled.second, scaled.scale2)):
+        if t is not None:
+            _need(t, "token_gate_pending output", torch.bfloat16)
+            _need(s, "token_gate_pending scale", torch.float32)
+            if tuple(t.shape) != tuple(h.shape) or s.shape[0] != width:
+                raise KernelError(f"token_gate_pending: output {tuple(t.shape)} with {s.shape[0]} factors, h {tuple(h.shape)}")
+    if h.shape[1] != width or tokens.shape[0] != h.shape[0] or column < 0 or column + dim > table.shape[1]:
+        raise KernelError(f"token_gate_pending: h {tuple(h.shape)}, weight {tuple(weight.shape)}, {tokens.shape[0]} tokens, columns "
+                          f"from {column} of a table {tuple(table.shape)}")
+    out = torch.empty((h.shape[0], dim), dtype=torch.bfloat16, device=h.device)
+    _call("thn_token_gate_product_bf16", _ptr(out), None, _ptr(h), _ptr(scaled.first), _ptr(scaled.scale1), _ptr(scaled.second),
+          _ptr(scaled.scale2 if scaled.second is not None else None), _ptr(weight), _ptr(table), _ptr(tokens), h.shape[0], width,
+          dim, table.shape[1], column, table.shape[0], _ptr(err), _stream())
+    return out
+
+
 def embed_norm(table: torch.Tensor, tokens: torch.Tensor, gain: Gain, err: Optional[torch.Tensor] = None,
                copy: bool = False) -> Tuple[torch.Tensor, Optional[torch.Tensor]]:
     """Token rows that pass an RMS norm as they start a float32 residual stream: ``gain(table[token])``.
@@ -648,8 +686,8 @@ def token_gate(x: torch.Tensor, weight: torch.Tensor, table: torch.Tensor, token
         raise KernelError("token_gate: the kernel with the product takes aligned bfloat16 rows of a multiple of eight entries")
     if can and (fused or (fused is None and x.shape[0] <= TOKEN_GATE_FUSED_ROWS)):
         out = torch.empty((x.shape[0], dim), dtype=x.dtype, device=x.device)
-        _call("thn_token_gate_product_bf16", _ptr(out), _ptr(x), _ptr(weight), _ptr(table), _ptr(tokens), x.shape[0], width, dim,
-              table.shape[1], column, table.shape[0], _ptr(err), _stream())
+        _call("thn_token_gate_product_bf16", _ptr(out), _ptr(x), None, None, None, None, None, _ptr(weight), _ptr(table),
+              _ptr(tokens), x.shape[0], width, dim, table.shape[1], column, table.shape[0], _ptr(err), _stream())
         return out
     z = linear(x, weight, err=err)
     out = torch.empty_like(z)
@@ -728,6 +766,7 @@ STREAM_MIN_N = 65536
 STREAM_POLICY = os.environ.get("THN_LINEAR_STREAM", "auto")     # auto | all | none (measurement)
 
 _device_counters = {}
+_counter_lane = 0       # 1 while work is issued to a second stream
 
 
 COUNTER_SLOTS = 1 << 20
@@ -736,15 +775,52 @@ COUNTER_SLOTS = 1 << 20
 def _counter_buffer(n: int, device) -> torch.Tensor:
     """Arrival counters for kernels whose last-arriving block finishes a shared result; zero
     between calls (the kernels reset them).  One buffer per device for the life of the
-    process: captured graphs hold its address, so it is never replaced by a larger one."""
-    if n > COUNTER_SLOTS:
-        raise KernelError(f"a kernel asks for {n} arrival counters, the buffer holds {COUNTER_SLOTS}")
+    process: captured graphs hold its address, so it is never replaced by a larger one.  Kernels that
+    run beside others (:class:`Beside`) have a part of it to themselves."""
+    if n > COUNTER_SLOTS // 2:
+        raise KernelError(f"a kernel asks for {n} arrival counters, the buffer holds {COUNTER_SLOTS // 2} for it")
     index = torch.device(device).index or 0
     have = _device_counters.get(index)
     if have is None:
         have = torch.zeros(COUNTER_SLOTS, dtype=torch.int32, device=device)
         _device_counters[index] = have
-    return have
+    return have[_counter_lane * (COUNTER_SLOTS // 2):]
+
+
+class Beside:
+    """A second stream for work that does not depend on what the current stream does next::
+
+        with beside:            # sees everything issued to the current stream so far
+            f = ...
+        a = ...                 # runs beside it
+        beside.join()           # the current stream waits for it
+
+    What the block allocates belongs to the second stream; the current stream may read it after ``join``
+    and until the next ``with``.  Works the same while a step is captured as a graph (the two become
+    branches of it).  Not to be nested."""
+
+    def __init__(self, device):
+        self.stream = torch.cuda.Stream(device)
+        self._inside = None
+
+    def __enter__(self):
+        global _counter_lane
+        if _counter_lane:
+            raise KernelError("work beside the current stream is not nested")
+        self.stream.wait_stream(torch.cuda.current_stream())
+        self._inside = torch.cuda.stream(self.stream)
+        self._inside.__enter__()
+        _counter_lane = 1
+        return self
+
+    def __exit__(self, *exc):
+        global _counter_lane
+        _counter_lane = 0
+        self._inside.__exit__(*exc)
+        return False
+
+    def join(self) -> None:
+        torch.cuda.current_stream().wait_stream(self.stream)
 
 
 _stream_needs = {}

@@ -169,12 +169,21 @@ class Attention:
             out[f"row_tiles/{size}/row0"], out[f"row_tiles/{size}/rows"] = ops.row_tiles_of(
                 batch.counts, batch.held, size)
 
-    def _out(self, a: torch.Tensor, proj: torch.Tensor, ctx: StepContext) -> torch.Tensor:
+    def _out(self, a: torch.Tensor, proj: torch.Tensor, ctx: StepContext, offset: int = 0) -> torch.Tensor:
         if self.gated:
-            a = ops.logistic_gate(a, proj, self.gate_offset, self.value_dim)
+            a = ops.logistic_gate(a, proj, offset + self.gate_offset, self.value_dim)
         return ops.linear(a, self.w_o, err=ctx.err)
 
     def forward(self, x: torch.Tensor, ctx: StepContext, entry: ScheduleEntry) -> torch.Tensor:
+        return self.forward_rows(ops.linear(x, self.w_qkv, err=ctx.err, bias=self.b_qkv), 0, ctx, entry)
+
+    def joint_rows(self):
+        return (self.w_qkv, self.b_qkv) if self.general and not self.shared_kv else None
+
+    def take_rows(self, weight: torch.Tensor, bias: Optional[torch.Tensor]) -> None:
+        self.w_qkv, self.b_qkv = weight, bias
+
+    def forward_rows(self, qkv: torch.Tensor, offset: int, ctx: StepContext, entry: ScheduleEntry) -> torch.Tensor:
         kv = ctx.cache.kv_view(entry.cache)
         tiles = None
         if ctx.rows.max_q_len > 1:
@@ -182,7 +191,6 @@ class Attention:
             row0 = ctx.inputs.get(f"row_tiles/{size}/row0") if size else None
             if row0 is not None:
                 tiles = ops.RowTiles(row0, ctx.inputs[f"row_tiles/{size}/rows"], row0.shape[0], size)
-        qkv = ops.linear(x, self.w_qkv, err=ctx.err, bias=self.b_qkv)
         if self.shared_kv:
             if entry.writes_cache:
                 raise ValueError("attention: a mixer without keys of its own cannot write a cache")
@@ -196,13 +204,13 @@ class Attention:
             rotary = self.position.tables() if self.position is not None else None
             if self.general:
                 q = ops.qk_prepare(qkv, self.q_gain, self.k_gain, self.norm_scope, self.eps or 1.0, rotary, ctx.rows, kv,
-                                   self.n_q, self.values_are_keys, entry.writes_cache, ctx.err)
+                                   self.n_q, self.values_are_keys, entry.writes_cache, ctx.err, proj_offset=offset)
             else:
                 q = ops.qk_norm_rope_cache(qkv, self.q_gain, self.k_gain, self.eps if self.eps is not None else 1.0,
                                            rotary, ctx.rows, kv, self.n_q, entry.writes_cache, ctx.err)
             a = ops.attention(q, ctx.rows, kv, self.n_q, self.scale, self.window, ctx.err, tiles, self.keep_first,
                               self.chunk, self.exact_weights, self.shape, self.sinks)
-            return self._out(a, qkv, ctx)
+            return self._out(a, qkv, ctx, offset)
         a = ops.qkv_attention(qkv, self.q_gain, self.k_gain, self.eps if self.eps is not None else 1.0,
                               self.position.tables() if self.position is not None else None,
                               ctx.rows, kv, self.n_q, self.scale, self.window, entry.writes_cache, ctx.err, tiles)

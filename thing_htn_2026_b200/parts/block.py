@@ -26,7 +26,10 @@ block, default 1; the feed-forward may be absent).  The two outputs travel as on
 the stream, norm of the sum" is one kernel at the next layer's norm or at the model's last.  With
 ``layer_scale`` (and the tensors ``mixer_scale`` and, beside a feed-forward, ``ffn_scale``, a vector each)
 it is ``y = x + s * mixer(n) + s' * ffn(n)``, entry by entry.  ``side``: a part that adds something of its own
-behind the sublayers, ``z = y + side(y)`` (:mod:`.side`).
+behind the sublayers, ``z = y + side(y)`` (:mod:`.side`).  Where both sublayers can work on a slice of wider
+projected rows (``joint_rows``: their input weight and bias, ``take_rows``: the same rows at their new place,
+``forward_rows``: from the projected rows on), ONE product serves them, and in single-token steps the
+feed-forward runs on a second stream beside the mixer (``THN_PARALLEL_STREAMS=0``: one after the other).
 
 ``hyper_connections``: the residual stream is ``streams`` copies ``X_0 .. X_(s-1)`` in float32,
 all equal to the embedding's row at the start.  A sublayer f with the numbers ``read[s]``,
@@ -41,6 +44,7 @@ Without the numbers' tensors (``connections`` False) it is one copy and the plai
 
 from __future__ import annotations
 
+import os
 from typing import Dict, List, Optional, Tuple
 
 import torch
@@ -49,8 +53,12 @@ from ..cache.sequence_cache import CacheNeed
 from ..config.base import PartSpec, ScheduleEntry
 from .. import ops
 from ..weights.loader import GAIN, TensorSpec
+from .fused import cat_bias, pad_rows
 from .registry import part_class, register_part
 from .runtime import Branch, HostBatch, Runtime, StepContext
+
+
+PARALLEL_STREAMS = os.environ.get("THN_PARALLEL_STREAMS", "1").strip().lower() not in ("0", "false", "no", "off")
 
 
 class Block:
@@ -172,6 +180,37 @@ class ParallelBlock(Block):
             self.mixer_scale = runtime.tensor(spec, "mixer_scale").to(torch.float32).contiguous()
             if self.ffn is not None:
                 self.ffn_scale = runtime.tensor(spec, "ffn_scale").to(torch.float32).contiguous()
+        self._join(runtime)
+
+    def _join(self, runtime: Runtime) -> None:
+        """One input product over the rows of both sublayers, where both can read a slice of its result."""
+        self.w_in = self.b_in = self.beside = None
+        rows = [part.joint_rows() if hasattr(part, "joint_rows") else None for part in (self.mixer, self.ffn)]
+        if any(r is None for r in rows) or rows[0][0].shape[0] % 8:
+            return
+        self.ffn_offset = at = rows[0][0].shape[0]
+        end = at + rows[1][0].shape[0]
+        rows[1] = (pad_rows(rows[1][0], at), rows[1][1])       # projected rows of whole 16-byte pieces
+        self.w_in, self.b_in = torch.cat([w for w, _ in rows], dim=0).contiguous(), cat_bias(rows)
+        # the members' own weights become slices of the joint one: nothing is held twice
+        self.mixer.take_rows(self.w_in[:at], None if rows[0][1] is None else self.b_in[:at])
+        self.ffn.take_rows(self.w_in[at:end], None if rows[1][1] is None else self.b_in[at:end])
+        if PARALLEL_STREAMS:
+            if "beside" not in runtime.shared:
+                runtime.shared["beside"] = ops.Beside(runtime.device)
+            self.beside = runtime.shared["beside"]
+
+    def _sublayers(self, n: torch.Tensor, ctx: StepContext, entry: ScheduleEntry):
+        if self.w_in is None:
+            return self.mixer.forward(n, ctx, entry), self.ffn.forward(n, ctx) if self.ffn is not None else None
+        proj = ops.linear(n, self.w_in, err=ctx.err, bias=self.b_in)
+        if self.beside is None or ctx.rows.max_q_len > 1:
+            return self.mixer.forward_rows(proj, 0, ctx, entry), self.ffn.forward_rows(proj, self.ffn_offset, ctx)
+        with self.beside:
+            f = self.ffn.forward_rows(proj, self.ffn_offset, ctx)
+        a = self.mixer.forward_rows(proj, 0, ctx, entry)
+        self.beside.join()
+        return a, f
 
     def forward(self, h: torch.Tensor, d, ctx: StepContext, entry: ScheduleEntry):
         if h.dtype != torch.float32:
@@ -182,14 +221,15 @@ class ParallelBlock(Block):
             n = self.norm.add_forward(h, d, post=d.norm)
         else:
             n = self.norm.add_forward(h, d)
-        a = self.mixer.forward(n, ctx, entry)
-        f = self.ffn.forward(n, ctx) if self.ffn is not None else None
+        a, f = self._sublayers(n, ctx, entry)
         if self.mixer_scale is not None:
             d = Branch(None, scaled=ops.ScaledPair(a, self.mixer_scale, f, self.ffn_scale))
         else:
             d = Branch(a, None, f, self.factor)
         if self.side is None:
             return h, d
+        if d.tensor is None and self.side.reads_pending(h):
+            return h, self.side.forward_pending(h, d, ctx)
         return h, self.side.forward(self.norm.add_read(h, d), ctx)
 
 

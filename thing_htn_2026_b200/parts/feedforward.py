@@ -85,10 +85,18 @@ class ClampedGLU:
         self.w_gate_up = torch.cat([runtime.tensor(spec, "gate_proj"), runtime.tensor(spec, "up_proj")], dim=0).contiguous()
         self.w_down = runtime.tensor(spec, "down_proj")
 
-    def forward(self, x: torch.Tensor, ctx) -> torch.Tensor:
+    def joint_rows(self):
+        return self.w_gate_up, None
+
+    def take_rows(self, weight: torch.Tensor, bias) -> None:
+        self.w_gate_up = weight
+
+    def forward_rows(self, proj: torch.Tensor, offset: int, ctx) -> torch.Tensor:
         err = getattr(ctx, "err", None)
-        y = ops.clamped_glu(ops.linear(x, self.w_gate_up, err=err), self.limit, self.slope)
-        return ops.linear(y, self.w_down, err=err)
+        return ops.linear(ops.clamped_glu(proj, self.limit, self.slope, offset, self.w_down.shape[1]), self.w_down, err=err)
+
+    def forward(self, x: torch.Tensor, ctx) -> torch.Tensor:
+        return self.forward_rows(ops.linear(x, self.w_gate_up, err=getattr(ctx, "err", None)), 0, ctx)
 
 
 @register_part("ffn", "routed_experts")

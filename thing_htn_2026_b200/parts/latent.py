@@ -148,7 +148,18 @@ class LatentAttention:
             out[f"row_tiles/{size}/row0"], out[f"row_tiles/{size}/rows"] = ops.row_tiles_of(
                 batch.counts, batch.held, size)
 
+    def joint_rows(self):
+        return self.w_in, None
+
+    def take_rows(self, weight: torch.Tensor, bias: Optional[torch.Tensor]) -> None:
+        if bias is not None:
+            raise ValueError("latent_attention: the input projections have no bias")
+        self.w_in = weight
+
     def forward(self, x: torch.Tensor, ctx: StepContext, entry: ScheduleEntry) -> torch.Tensor:
+        return self.forward_rows(ops.linear(x, self.w_in, err=ctx.err), 0, ctx, entry)
+
+    def forward_rows(self, proj: torch.Tensor, offset: int, ctx: StepContext, entry: ScheduleEntry) -> torch.Tensor:
         kv = ctx.cache.kv_view(entry.cache)
         tiles = None
         if ctx.rows.max_q_len > 1:
@@ -156,19 +167,18 @@ class LatentAttention:
             row0 = ctx.inputs.get(f"row_tiles/{size}/row0") if size else None
             if row0 is not None:
                 tiles = ops.RowTiles(row0, ctx.inputs[f"row_tiles/{size}/rows"], row0.shape[0], size)
-        proj = ops.linear(x, self.w_in, err=ctx.err)
         q_rows = None
         if self.q_rank:
-            q_latent, latent = ops.latent_norm(proj, 0, self.q_rank, self.q_gain, self.eps,
-                                               second=(self.latent_offset, self.rank, self.latent_gain))
+            q_latent, latent = ops.latent_norm(proj, offset, self.q_rank, self.q_gain, self.eps,
+                                               second=(offset + self.latent_offset, self.rank, self.latent_gain))
             q_rows = ops.linear(q_latent, self.w_uq, err=ctx.err)
         else:
-            latent = ops.latent_norm(proj, self.latent_offset, self.rank, self.latent_gain, self.eps)
+            latent = ops.latent_norm(proj, offset + self.latent_offset, self.rank, self.latent_gain, self.eps)
         up = ops.linear(latent, self.w_up, err=ctx.err)
-        q = ops.latent_assemble(proj, 0, self.shared_offset, up, self.position.tables() if self.position else None,
+        q = ops.latent_assemble(proj, 0 if self.q_rank else offset, offset + self.shared_offset, up, self.position.tables() if self.position else None,
                                 ctx.rows, kv, self.n_heads, self.plain, self.rot, ctx.err, self.value_dim, q_rows)
         a = ops.attention(q, ctx.rows, kv, self.n_heads, self.scale, self.window, ctx.err, tiles,
                           exact_weights=self.exact_weights, sinks=self.sinks)
         if self.gated:
-            a = ops.logistic_gate(a, proj, self.gate_offset, self.out_dim if self.head_gate else 1)
+            a = ops.logistic_gate(a, proj, offset + self.gate_offset, self.out_dim if self.head_gate else 1)
         return ops.linear(a, self.w_o, err=ctx.err)

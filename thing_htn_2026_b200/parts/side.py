@@ -7,10 +7,12 @@ type), t the row's token and ``dim`` columns of a table that all layers share, s
     y = W_proj g,     x <- x + norm(y)
 
 The norm is a part of its own; its output is added by the kernel that also computes the next layer's norm
-(the result travels as a :class:`Branch`).  Kernels: csrc/token_side.cu."""
+(the result travels as a :class:`Branch`).  In steps of few rows the gate's kernel reads the stream and what is
+pending on it, so that no kernel of its own has to add that first.  Kernels: csrc/token_side.cu."""
 
 from __future__ import annotations
 
+from dataclasses import replace
 from typing import List
 
 import torch
@@ -47,3 +49,13 @@ class TokenRows:
     def forward(self, x: torch.Tensor, ctx: StepContext) -> Branch:
         g = ops.token_gate(x, self.w_gate, self.table, ctx.tokens, self.column, err=ctx.err)
         return Branch(ops.linear(g, self.w_proj, err=ctx.err), self.norm)
+
+    def reads_pending(self, h: torch.Tensor) -> bool:
+        """Whether ``forward_pending`` serves a step of these rows."""
+        return h.shape[0] <= ops.TOKEN_GATE_FUSED_ROWS and ops.token_gate_pending_supported(h, self.w_gate)
+
+    def forward_pending(self, h: torch.Tensor, d: Branch, ctx: StepContext) -> Branch:
+        """The same from the stream and the scaled outputs that are still to be added to it: they are added
+        in the gate's kernel for what it reads, and to the stream itself together with this part's output."""
+        g = ops.token_gate_pending(h, d.scaled, self.w_gate, self.table, ctx.tokens, self.column, err=ctx.err)
+        return replace(d, tensor=ops.linear(g, self.w_proj, err=ctx.err), norm=self.norm)
