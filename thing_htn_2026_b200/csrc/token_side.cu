@@ -108,11 +108,6 @@ __global__ void __launch_bounds__(kProductThreads) token_gate_product_kernel(
     const __nv_bfloat16* __restrict__ table, const int* __restrict__ tokens, int dim, int vecs, long long table_width,
     int column0, int n_table_rows, int* __restrict__ err) {
     pdl_launch_dependents();
-    // the weight's rows of this block, into L2 while the kernel before still runs
-    for (int n0 = blockIdx.y * 4; n0 < dim; n0 += gridDim.y * 4)
-        for (int j = 0; j < 4 && n0 + j < dim; ++j)
-            for (int i = threadIdx.x * 8; i < vecs; i += kProductThreads * 8)
-                asm volatile("prefetch.global.L2 [%0];" ::"l"(reinterpret_cast<const uint4*>(w) + (size_t)(n0 + j) * vecs + i));
     pdl_wait();
     extern __shared__ uint4 row[];          // PENDING: the row, rounded
     __shared__ float part[kProductThreads / 32][4];
